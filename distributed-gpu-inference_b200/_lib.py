@@ -214,6 +214,46 @@ MIXER_SIGNATURES = {
     "b200_router_logits": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_void_p]),
     "b200_gated_table_rows": (
         c_int, [c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_int, c_void_p, c_int64, c_int, c_int, c_void_p]),
+    # one decay per token and head, dynamic tanh norms, sigmoid group routing (csrc/b200_recurrent_ops.cu)
+    "b200_causal_conv_silu_ext": (
+        c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
+                c_int, c_int, c_int, c_void_p]),
+    "b200_latent_rotary_append_ext": (
+        c_int, [c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int64, c_void_p, c_int64, c_void_p,
+                c_float, c_void_p, c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
+                c_int, c_int, c_void_p]),
+    "b200_router_logits_ext": (
+        c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_void_p]),
+    "b200_group_topk": (
+        c_int, [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int, c_int, c_int, c_float, c_float,
+                c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "b200_residual_dyn_tanh": (
+        c_int, [c_void_p, c_void_p, c_int64, c_int, c_void_p, c_void_p, c_float, c_void_p, c_int64, c_int,
+                c_int, c_void_p]),
+    "b200_expert_combine_dyn_tanh": (
+        c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_int64, c_void_p,
+                c_void_p, c_float, c_void_p, c_int64, c_int, c_int, c_void_p]),
+    "b200_silu_glu": (
+        c_int, [c_void_p, c_void_p, c_int64, c_int, c_int, c_void_p]),
+    "b200_capped_gates": (
+        c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_float,
+                c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
+    "b200_step_sizes": (
+        c_int, [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int, c_int, c_void_p]),
+    "b200_decay_scan": (
+        c_int, [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
+                c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                c_int, c_int, c_void_p]),
+    "b200_decay_step": (
+        c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64,
+                c_int, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_float, c_void_p, c_float,
+                c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "b200_normalized_head_out": (
+        c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int64,
+                c_float, c_void_p, c_void_p, c_int64, c_int, c_int, c_int, c_void_p]),
+    "b200_gated_part_norm": (
+        c_int, [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_float, c_int64, c_int, c_int, c_int,
+                c_void_p]),
 }
 
 _lock = threading.Lock()
@@ -269,7 +309,7 @@ def _build_mixers() -> None:
         fcntl.flock(lock, fcntl.LOCK_EX)
         if os.path.exists(MIXER_LIB_PATH):
             return
-        proc = subprocess.run(["make", "-j4", "-C", csrc, "mixers"], stdout=subprocess.PIPE, stderr=subprocess.STDOUT)
+        proc = subprocess.run(["make", "-j5", "-C", csrc, "mixers"], stdout=subprocess.PIPE, stderr=subprocess.STDOUT)
         if proc.returncode != 0 or not os.path.exists(MIXER_LIB_PATH):
             raise B200LibraryError("building libb200_mixers.so failed:\n" + proc.stdout.decode(errors="replace")[-4000:])
 

@@ -101,7 +101,7 @@ latent_rotary_append_kernel(const T* __restrict__ q_rot, int64_t q_tok_stride, i
                             int64_t qo_tok_stride, int64_t qo_head_stride, const T* __restrict__ dkv, int64_t dkv_stride,
                             const T* __restrict__ w_c, float eps, const double* __restrict__ freqs, float gain, int rot_dims,
                             T* __restrict__ pool, const int64_t* __restrict__ slot_mapping,
-                            const int32_t* __restrict__ tok_pos, int H, int dr, int rank) {
+                            const int32_t* __restrict__ tok_pos, int H, int dr, int rank, int interleaved) {
   extern __shared__ float cs[];   // [rot_dims / 2][2]
   __shared__ float red[32];
   const int64_t n = blockIdx.x;
@@ -113,6 +113,16 @@ latent_rotary_append_kernel(const T* __restrict__ q_rot, int64_t q_tok_stride, i
     cs[2 * i] = static_cast<float>(c) * gain;
     cs[2 * i + 1] = static_cast<float>(s) * gain;
   }
+  // column i < rot_dims of a rotated part: its partner, its pair, and whether it is the pair's second member
+  auto turn = [&](const T* part, int i) -> float {
+    const float y = Cvt<T>::to_f32(part[i]);
+    if (i >= rot_dims) return y;
+    const bool second = interleaved ? (i & 1) : i >= half;
+    const int pair = interleaved ? i >> 1 : (second ? i - half : i);
+    const float other = Cvt<T>::to_f32(part[interleaved ? i ^ 1 : (second ? i - half : i + half)]);
+    const float c = cs[2 * pair], s = cs[2 * pair + 1];
+    return second ? fmaf(y, c, other * s) : fmaf(y, c, -other * s);   // (u, v) -> (u c - v s, v c + u s)
+  };
   const T* row = dkv + n * dkv_stride;
   float ss = 0.f;
   for (int i = threadIdx.x; i < rank; i += blockDim.x) {
@@ -125,27 +135,13 @@ latent_rotary_append_kernel(const T* __restrict__ q_rot, int64_t q_tok_stride, i
     T* dst = pool + slot * (rank + dr);
     for (int i = threadIdx.x; i < rank; i += blockDim.x)
       dst[i] = Cvt<T>::from_f32(Cvt<T>::to_f32(row[i]) * inv * Cvt<T>::to_f32(w_c[i]));
-    for (int i = threadIdx.x; i < dr; i += blockDim.x) {
-      float y = Cvt<T>::to_f32(row[rank + i]);
-      if (i < rot_dims) {
-        const float other = Cvt<T>::to_f32(row[rank + (i ^ 1)]);
-        const float c = cs[i & ~1], s = cs[i | 1];
-        y = (i & 1) ? fmaf(y, c, other * s) : fmaf(y, c, -other * s);   // (u, v) -> (u c - v s, v c + u s)
-      }
-      dst[rank + i] = Cvt<T>::from_f32(y);
-    }
+    for (int i = threadIdx.x; i < dr; i += blockDim.x) dst[rank + i] = Cvt<T>::from_f32(turn(row + rank, i));
   }
   const T* qs = q_rot + n * q_tok_stride;
   T* qd = q_out + n * qo_tok_stride;
   for (int e = threadIdx.x; e < H * dr; e += blockDim.x) {
     const int h = e / dr, i = e - h * dr;
-    float y = Cvt<T>::to_f32(qs[h * q_head_stride + i]);
-    if (i < rot_dims) {
-      const float other = Cvt<T>::to_f32(qs[h * q_head_stride + (i ^ 1)]);
-      const float c = cs[i & ~1], s = cs[i | 1];
-      y = (i & 1) ? fmaf(y, c, other * s) : fmaf(y, c, -other * s);
-    }
-    qd[h * qo_head_stride + i] = Cvt<T>::from_f32(y);
+    qd[h * qo_head_stride + i] = Cvt<T>::from_f32(turn(qs + h * q_head_stride, i));
   }
 }
 
@@ -256,54 +252,85 @@ gated_table_rows_kernel(T* __restrict__ out, const T* __restrict__ z, int64_t z_
 }
 
 // ---- router logits -------------------------------------------------------------------------------------------------
-// One CTA of four warps per token, kRouterChunk experts at a time: thread t owns columns t, t + 128, ... (four at a time
+// One CTA of four warps per token (or per few tokens), kRouterChunk experts at a time: thread t owns columns t, t + 128, ... (four at a time
 // when the width allows); partial sums meet in a butterfly per warp and the four warps' sums are added in warp order.
 // The order of every sum depends on the width alone, so a token's logits - and with them its experts - do not depend on
 // what else the step carries.
 constexpr int kRouterChunk = 8;
 constexpr int kRouterThreads = 128;
 
-template <bool VEC>
+template <typename X>
+__device__ __forceinline__ float4 row4(const X* p) {
+  if constexpr (sizeof(X) == 4) {
+    return *reinterpret_cast<const float4*>(p);
+  } else {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const X* e = reinterpret_cast<const X*>(&raw);
+    return make_float4(Cvt<X>::to_f32(e[0]), Cvt<X>::to_f32(e[1]), Cvt<X>::to_f32(e[2]), Cvt<X>::to_f32(e[3]));
+  }
+}
+
+// TOK tokens per CTA share every weight that is read (steps of many tokens); a token's own sums do not see the others.
+template <typename X, bool VEC, int TOK>
 __global__ void __launch_bounds__(kRouterThreads)
-router_logits_kernel(float* __restrict__ logits, const float* __restrict__ x, const float* __restrict__ w,
-                     const float* __restrict__ bias, int E, int W) {
-  __shared__ float part[kRouterThreads / 32][kRouterChunk];
-  const int64_t n = blockIdx.x;
+router_logits_kernel(float* __restrict__ logits, const X* __restrict__ x, const float* __restrict__ w,
+                     const float* __restrict__ bias, int64_t n_tok, int E, int W) {
+  __shared__ float part[kRouterThreads / 32][TOK][kRouterChunk];
+  const int64_t n0 = static_cast<int64_t>(blockIdx.x) * TOK;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const float* xr = x + n * W;
-  for (int e0 = 0; e0 < E; e0 += kRouterChunk) {
-    float acc[kRouterChunk];
+  const X* xr[TOK];
 #pragma unroll
-    for (int j = 0; j < kRouterChunk; ++j) acc[j] = 0.f;
+  for (int t = 0; t < TOK; ++t) xr[t] = x + (n0 + t < n_tok ? n0 + t : n0) * W;
+  for (int e0 = 0; e0 < E; e0 += kRouterChunk) {
+    float acc[TOK][kRouterChunk];
+#pragma unroll
+    for (int t = 0; t < TOK; ++t)
+#pragma unroll
+      for (int j = 0; j < kRouterChunk; ++j) acc[t][j] = 0.f;
     if (VEC) {
       for (int i = threadIdx.x * 4; i < W; i += kRouterThreads * 4) {
-        const float4 xv = *reinterpret_cast<const float4*>(xr + i);
+        float4 xv[TOK];
+#pragma unroll
+        for (int t = 0; t < TOK; ++t) xv[t] = row4(xr[t] + i);
 #pragma unroll
         for (int j = 0; j < kRouterChunk; ++j)
           if (e0 + j < E) {
             const float4 wv = *reinterpret_cast<const float4*>(w + static_cast<int64_t>(e0 + j) * W + i);
-            acc[j] = fmaf(xv.x, wv.x, fmaf(xv.y, wv.y, fmaf(xv.z, wv.z, fmaf(xv.w, wv.w, acc[j]))));
+#pragma unroll
+            for (int t = 0; t < TOK; ++t)
+              acc[t][j] = fmaf(xv[t].x, wv.x, fmaf(xv[t].y, wv.y, fmaf(xv[t].z, wv.z, fmaf(xv[t].w, wv.w, acc[t][j]))));
           }
       }
     } else {
       for (int i = threadIdx.x; i < W; i += kRouterThreads) {
-        const float xv = xr[i];
+        float xv[TOK];
+#pragma unroll
+        for (int t = 0; t < TOK; ++t) xv[t] = Cvt<X>::to_f32(xr[t][i]);
 #pragma unroll
         for (int j = 0; j < kRouterChunk; ++j)
-          if (e0 + j < E) acc[j] = fmaf(xv, w[static_cast<int64_t>(e0 + j) * W + i], acc[j]);
+          if (e0 + j < E) {
+            const float wv = w[static_cast<int64_t>(e0 + j) * W + i];
+#pragma unroll
+            for (int t = 0; t < TOK; ++t) acc[t][j] = fmaf(xv[t], wv, acc[t][j]);
+          }
       }
     }
 #pragma unroll
-    for (int j = 0; j < kRouterChunk; ++j) {
-      const float t = warp_sum(acc[j]);
-      if (lane == 0) part[warp][j] = t;
-    }
-    __syncthreads();
-    if (threadIdx.x < kRouterChunk && e0 + threadIdx.x < E) {
-      float t = part[0][threadIdx.x];
+    for (int t = 0; t < TOK; ++t)
 #pragma unroll
-      for (int ww = 1; ww < kRouterThreads / 32; ++ww) t += part[ww][threadIdx.x];
-      logits[n * E + e0 + threadIdx.x] = t + (bias ? bias[e0 + threadIdx.x] : 0.f);
+      for (int j = 0; j < kRouterChunk; ++j) {
+        const float s = warp_sum(acc[t][j]);
+        if (lane == 0) part[warp][t][j] = s;
+      }
+    __syncthreads();
+    if (threadIdx.x < TOK * kRouterChunk) {
+      const int t = threadIdx.x / kRouterChunk, j = threadIdx.x % kRouterChunk;
+      if (e0 + j < E && n0 + t < n_tok) {
+        float s = part[0][t][j];
+#pragma unroll
+        for (int ww = 1; ww < kRouterThreads / 32; ++ww) s += part[ww][t][j];
+        logits[(n0 + t) * E + e0 + j] = s + (bias ? bias[e0 + j] : 0.f);
+      }
     }
     __syncthreads();
   }
@@ -336,6 +363,16 @@ int b200_latent_rotary_append(const void* q_rot, int64_t q_tok_stride, int64_t q
                               const void* c_norm, float eps, const double* freqs, float gain, int rot_dims, void* pool,
                               const int64_t* slot_mapping, const int32_t* tok_pos, int n_tok, int H, int rot_width,
                               int rank, int dtype, void* stream) {
+  return b200_latent_rotary_append_ext(q_rot, q_tok_stride, q_head_stride, q_out, qo_tok_stride, qo_head_stride, dkv,
+                                       dkv_stride, c_norm, eps, freqs, gain, rot_dims, 1, pool, slot_mapping, tok_pos, n_tok,
+                                       H, rot_width, rank, dtype, stream);
+}
+
+int b200_latent_rotary_append_ext(const void* q_rot, int64_t q_tok_stride, int64_t q_head_stride, void* q_out,
+                                  int64_t qo_tok_stride, int64_t qo_head_stride, const void* dkv, int64_t dkv_stride,
+                                  const void* c_norm, float eps, const double* freqs, float gain, int rot_dims,
+                                  int interleaved, void* pool, const int64_t* slot_mapping, const int32_t* tok_pos, int n_tok,
+                                  int H, int rot_width, int rank, int dtype, void* stream) {
   if (n_tok < 0 || H <= 0 || rot_width < 0 || rank <= 0 || rot_dims < 0 || rot_dims > rot_width || (rot_dims & 1))
     return fail(B200_EINVAL, "b200_latent_rotary_append: bad sizes");
   if (n_tok == 0) return 0;
@@ -347,7 +384,7 @@ int b200_latent_rotary_append(const void* q_rot, int64_t q_tok_stride, int64_t q
     latent_rotary_append_kernel<T><<<n_tok, 128, smem, static_cast<cudaStream_t>(stream)>>>(
         static_cast<const T*>(q_rot), q_tok_stride, q_head_stride, static_cast<T*>(q_out), qo_tok_stride, qo_head_stride,
         static_cast<const T*>(dkv), dkv_stride, static_cast<const T*>(c_norm), eps, freqs, gain, rot_dims,
-        static_cast<T*>(pool), slot_mapping, tok_pos, H, rot_width, rank);
+        static_cast<T*>(pool), slot_mapping, tok_pos, H, rot_width, rank, interleaved);
     return check_launch("b200_latent_rotary_append");
   });
 }
@@ -431,16 +468,30 @@ int b200_gated_table_rows(void* out, const void* z, int64_t z_stride, const void
 
 int b200_router_logits(float* logits, const float* x, const float* w, const float* bias, int64_t n_tok, int E, int width,
                        void* stream) {
+  return b200_router_logits_ext(logits, x, w, bias, n_tok, E, width, B200_DTYPE_F32, stream);
+}
+
+int b200_router_logits_ext(float* logits, const void* x, const float* w, const float* bias, int64_t n_tok, int E, int width,
+                           int dtype, void* stream) {
   if (n_tok < 0 || E <= 0 || width <= 0) return fail(B200_EINVAL, "b200_router_logits: bad sizes");
   if (n_tok == 0) return 0;
   if (!logits || !x || !w) return fail(B200_EINVAL, "b200_router_logits: null pointer");
-  const unsigned grid = static_cast<unsigned>(n_tok);
-  auto s = static_cast<cudaStream_t>(stream);
-  if (width % 4 == 0 && aligned16(x) && aligned16(w))
-    router_logits_kernel<true><<<grid, kRouterThreads, 0, s>>>(logits, x, w, bias, E, width);
-  else
-    router_logits_kernel<false><<<grid, kRouterThreads, 0, s>>>(logits, x, w, bias, E, width);
-  return check_launch("b200_router_logits");
+  constexpr int kTok = 4;
+  const bool many = n_tok >= 4 * kTok * kNumSMs;
+  const unsigned grid = static_cast<unsigned>(many ? (n_tok + kTok - 1) / kTok : n_tok);
+  const bool vec = width % 4 == 0 && aligned16(x) && aligned16(w);
+  return gated_by_dtype(dtype, "b200_router_logits", [&](auto* tag) {
+    using X = std::remove_pointer_t<decltype(tag)>;
+    auto launch = [&](auto kern) {
+      kern<<<grid, kRouterThreads, 0, static_cast<cudaStream_t>(stream)>>>(logits, static_cast<const X*>(x), w, bias, n_tok, E,
+                                                                           width);
+    };
+    if (vec && many) launch(router_logits_kernel<X, true, kTok>);
+    else if (vec) launch(router_logits_kernel<X, true, 1>);
+    else if (many) launch(router_logits_kernel<X, false, kTok>);
+    else launch(router_logits_kernel<X, false, 1>);
+    return check_launch("b200_router_logits");
+  });
 }
 
 }  // extern "C"

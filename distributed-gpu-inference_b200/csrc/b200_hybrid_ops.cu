@@ -975,53 +975,105 @@ struct SeqSpan {
 
 constexpr int kConvTokens = 64;   // tokens per CTA; at least taps - 1, so only a sequence's first CTA reads the carried inputs
 
-template <typename T>
+template <typename T, int V>
+__device__ __forceinline__ void conv_load(float (&dst)[V], const T* p) {
+  if constexpr (V == 4) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+    for (int u = 0; u < 4; ++u) dst[u] = Cvt<T>::to_f32(e[u]);
+  } else {
+    dst[0] = Cvt<T>::to_f32(p[0]);
+  }
+}
+
+template <typename T, int TAPS, int V>
 __global__ void __launch_bounds__(128)
 causal_conv_silu_kernel(T* __restrict__ out, int64_t out_stride, const T* __restrict__ x, int64_t x_stride,
-                        const T* __restrict__ w, float* __restrict__ tail, const SeqSpan* __restrict__ seqs, int C,
-                        int taps) {
+                        const T* __restrict__ w, const T* __restrict__ bias, float* __restrict__ tail,
+                        const SeqSpan* __restrict__ seqs, int C, int taps) {
   const SeqSpan sq = seqs[blockIdx.x];
   const int t0 = blockIdx.y * kConvTokens;
   if (t0 >= sq.count) return;
-  const int c = blockIdx.z * blockDim.x + threadIdx.x;
+  const int c = (blockIdx.z * blockDim.x + threadIdx.x) * V;
   if (c >= C) return;
-  constexpr int kMaxTaps = 8;
-  float wr[kMaxTaps], old[kMaxTaps];
+  // slot i of a window is tap i - (TAPS - taps); slots before tap 0 carry weight 0 and are never loaded
+  const int pad = TAPS - taps;
+  float wr[TAPS][V], b[V], win[TAPS][V];
 #pragma unroll
-  for (int i = 0; i < kMaxTaps; ++i) {
-    wr[i] = i < taps ? Cvt<T>::to_f32(w[static_cast<int64_t>(c) * taps + i]) : 0.f;
-    old[i] = 0.f;
-  }
+  for (int i = 0; i < TAPS; ++i)
+#pragma unroll
+    for (int u = 0; u < V; ++u) {
+      wr[i][u] = i >= pad ? Cvt<T>::to_f32(w[static_cast<int64_t>(c + u) * taps + i - pad]) : 0.f;
+      win[i][u] = 0.f;
+    }
+#pragma unroll
+  for (int u = 0; u < V; ++u) b[u] = bias ? Cvt<T>::to_f32(bias[c + u]) : 0.f;
   float* tl = tail + static_cast<int64_t>(sq.slot) * (taps - 1) * C + c;   // [taps - 1][C], oldest first
-  if (t0 == 0 && !sq.fresh)
-#pragma unroll
-    for (int i = 0; i < kMaxTaps - 1; ++i)
-      if (i < taps - 1) old[i] = tl[static_cast<int64_t>(i) * C];
   const T* xc = x + static_cast<int64_t>(sq.tok0) * x_stride + c;
-  auto input = [&](int t) -> float {    // the channel's input at step t of this portion; t < 0 reaches into the carry
-    if (t >= 0) return Cvt<T>::to_f32(xc[static_cast<int64_t>(t) * x_stride]);
-    float r = 0.f;
+  // the window before token t0: slots 0 .. TAPS - 2 hold its last inputs, out of the carry where the portion has none
+  const bool carried = t0 == 0 && !sq.fresh;
 #pragma unroll
-    for (int i = 0; i < kMaxTaps - 1; ++i)
-      if (i == taps - 1 + t) r = old[i];
-    return r;
-  };
+  for (int i = 0; i < TAPS - 1; ++i) {
+    if (i < pad) continue;
+    const int t = t0 - (TAPS - 1) + i;
+    if (t >= 0) conv_load<T, V>(win[i], xc + static_cast<int64_t>(t) * x_stride);
+    else if (carried)
+#pragma unroll
+      for (int u = 0; u < V; ++u) win[i][u] = tl[static_cast<int64_t>(i - pad) * C + u];
+  }
+  float first[TAPS][V];                       // the carry itself, for the update below
+#pragma unroll
+  for (int i = 0; i < TAPS; ++i)
+#pragma unroll
+    for (int u = 0; u < V; ++u) first[i][u] = win[i][u];
   const int t1 = min(sq.count, t0 + kConvTokens);
+#pragma unroll 4
   for (int t = t0; t < t1; ++t) {
-    float y = 0.f;
+    conv_load<T, V>(win[TAPS - 1], xc + static_cast<int64_t>(t) * x_stride);
+    float y[V];
 #pragma unroll
-    for (int i = 0; i < kMaxTaps; ++i)
-      if (i < taps) y = fmaf(wr[i], input(t - (taps - 1 - i)), y);
-    out[static_cast<int64_t>(sq.tok0 + t) * out_stride + c] = Cvt<T>::from_f32(y * sigmoid_(y));
+    for (int u = 0; u < V; ++u) {
+      y[u] = 0.f;
+#pragma unroll
+      for (int i = 0; i < TAPS; ++i) y[u] = fmaf(wr[i][u], win[i][u], y[u]);
+      y[u] += b[u];
+      y[u] *= sigmoid_(y[u]);
+#pragma unroll
+      for (int i = 0; i < TAPS - 1; ++i) win[i][u] = win[i + 1][u];
+    }
+    T* dst = out + static_cast<int64_t>(sq.tok0 + t) * out_stride + c;
+    if constexpr (V == 4) {
+      uint2 raw;
+      T* e = reinterpret_cast<T*>(&raw);
+#pragma unroll
+      for (int u = 0; u < 4; ++u) e[u] = Cvt<T>::from_f32(y[u]);
+      *reinterpret_cast<uint2*>(dst) = raw;
+    } else {
+      dst[0] = Cvt<T>::from_f32(y[0]);
+    }
   }
   if (t0 == 0) {
     // the new carry: the portion's last taps - 1 inputs (older ones come from the old carry when the portion is short)
-    float nw[kMaxTaps];
 #pragma unroll
-    for (int i = 0; i < kMaxTaps - 1; ++i) nw[i] = (i < taps - 1) ? input(sq.count - (taps - 1) + i) : 0.f;
+    for (int i = 0; i < TAPS - 1; ++i) {
+      if (i < pad) continue;
+      const int t = sq.count - (TAPS - 1) + i;
+      float nw[V];
+      if (t >= 0) {
+        conv_load<T, V>(nw, xc + static_cast<int64_t>(t) * x_stride);
+      } else {                                // slot TAPS - 1 + t of the window before token 0
 #pragma unroll
-    for (int i = 0; i < kMaxTaps - 1; ++i)
-      if (i < taps - 1) tl[static_cast<int64_t>(i) * C] = nw[i];
+        for (int u = 0; u < V; ++u) {
+          nw[u] = 0.f;
+#pragma unroll
+          for (int j = 0; j < TAPS - 1; ++j)
+            if (j == TAPS - 1 + t) nw[u] = first[j][u];
+        }
+      }
+#pragma unroll
+      for (int u = 0; u < V; ++u) tl[static_cast<int64_t>(i - pad) * C + u] = nw[u];
+    }
   }
 }
 
@@ -1492,16 +1544,42 @@ int b200_mixed_prompt_attn_ext(void* out, int64_t out_tok_stride, int64_t out_he
 
 int b200_causal_conv_silu(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* w, float* tail,
                           const int32_t* seqs, int n_seqs, int max_count, int C, int taps, int dtype, void* stream) {
+  return b200_causal_conv_silu_ext(out, out_stride, x, x_stride, w, nullptr, tail, seqs, n_seqs, max_count, C, taps, dtype,
+                                   stream);
+}
+
+int b200_causal_conv_silu_ext(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* w, const void* bias,
+                              float* tail, const int32_t* seqs, int n_seqs, int max_count, int C, int taps, int dtype,
+                              void* stream) {
   if (n_seqs < 0 || C <= 0 || taps < 1 || max_count < 0) return fail(B200_EINVAL, "b200_causal_conv_silu: bad sizes");
-  if (taps > 8) return fail(B200_ESHAPE, "b200_causal_conv_silu: %d taps beyond 8", taps);
+  if (taps > 16) return fail(B200_ESHAPE, "b200_causal_conv_silu: %d taps beyond 16", taps);
   if (n_seqs == 0 || max_count == 0) return 0;
   if (!out || !x || !w || !seqs || (taps > 1 && !tail)) return fail(B200_EINVAL, "b200_causal_conv_silu: null pointer");
-  const dim3 grid(n_seqs, (max_count + kConvTokens - 1) / kConvTokens, (C + 127) / 128);
+  // four channels per thread (8-byte accesses) for 16-bit rows that allow it
+  const bool vec = dtype_size(dtype) == 2 && taps <= 8 && C % 4 == 0 && x_stride % 4 == 0 && out_stride % 4 == 0 &&
+                   (reinterpret_cast<uintptr_t>(x) & 7u) == 0 && (reinterpret_cast<uintptr_t>(out) & 7u) == 0;
+  const int per = vec ? 512 : 128;
+  const dim3 grid(n_seqs, (max_count + kConvTokens - 1) / kConvTokens, (C + per - 1) / per);
   return hybrid_by_dtype(dtype, "b200_causal_conv_silu", [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
-    causal_conv_silu_kernel<T><<<grid, 128, 0, static_cast<cudaStream_t>(stream)>>>(
-        static_cast<T*>(out), out_stride, static_cast<const T*>(x), x_stride, static_cast<const T*>(w), tail,
-        reinterpret_cast<const SeqSpan*>(seqs), C, taps);
+    auto launch = [&](auto kern) {
+      kern<<<grid, 128, 0, static_cast<cudaStream_t>(stream)>>>(
+          static_cast<T*>(out), out_stride, static_cast<const T*>(x), x_stride, static_cast<const T*>(w),
+          static_cast<const T*>(bias), tail, reinterpret_cast<const SeqSpan*>(seqs), C, taps);
+    };
+    if constexpr (sizeof(T) == 2) {
+      if (vec && taps <= 4) {
+        launch(causal_conv_silu_kernel<T, 4, 4>);
+        return check_launch("b200_causal_conv_silu");
+      }
+      if (vec) {
+        launch(causal_conv_silu_kernel<T, 8, 4>);
+        return check_launch("b200_causal_conv_silu");
+      }
+    }
+    if (taps <= 4) launch(causal_conv_silu_kernel<T, 4, 1>);
+    else if (taps <= 8) launch(causal_conv_silu_kernel<T, 8, 1>);
+    else launch(causal_conv_silu_kernel<T, 16, 1>);
     return check_launch("b200_causal_conv_silu");
   });
 }

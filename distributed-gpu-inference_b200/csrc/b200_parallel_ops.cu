@@ -426,7 +426,7 @@ cast_rows_kernel(T* __restrict__ out, const float* __restrict__ x, int64_t n) {
     out[i] = Cvt<T>::from_f32(x[i]);
 }
 
-// ---- grouped softmax routing ------------------------------------------------------------------------------------------
+// ---- grouped routing: softmax or sigmoid scores ------------------------------------------------------------------------------------------
 // One warp per token.  Shared memory per warp: score[E], choice[E], group best[groups].  Ties go to the lowest index.
 constexpr int kRouteWarps = 4;
 
@@ -443,9 +443,9 @@ __device__ __forceinline__ void warp_argmax(float& best, int& bi) {
 }
 
 __global__ void __launch_bounds__(kRouteWarps * 32)
-softmax_group_topk_kernel(int32_t* __restrict__ ids, float* __restrict__ weights, const float* __restrict__ logits,
-                          const float* __restrict__ correction, float sum_floor, int n_tok, int E, int top, int groups,
-                          int keep) {
+group_topk_kernel(int32_t* __restrict__ ids, float* __restrict__ weights, const float* __restrict__ logits,
+                  int64_t logit_stride, const float* __restrict__ correction, int sigmoid_scores, int group_best,
+                  int normalize, float sum_floor, float weight_scale, int n_tok, int E, int top, int groups, int keep) {
   extern __shared__ float rt_sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int tok = blockIdx.x * kRouteWarps + warp;
@@ -453,30 +453,47 @@ softmax_group_topk_kernel(int32_t* __restrict__ ids, float* __restrict__ weights
   float* score = rt_sm + warp * (2 * E + groups);
   float* choice = score + E;
   float* gbest = choice + E;
-  const float* z = logits + static_cast<int64_t>(tok) * E;
-  float m = -INFINITY;
-  for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
-  m = warp_max(m);
-  float sum = 0.f;
-  for (int e = lane; e < E; e += 32) {
-    const float x = expf(z[e] - m);
-    score[e] = x;
-    sum += x;
-  }
-  sum = warp_sum(sum);
-  for (int e = lane; e < E; e += 32) {
-    const float s = score[e] / sum;
-    score[e] = s;
-    choice[e] = s + (correction ? correction[e] : 0.f);
+  const float* z = logits + static_cast<int64_t>(tok) * logit_stride;
+  if (sigmoid_scores) {
+    for (int e = lane; e < E; e += 32) {
+      const float s = sigm(z[e]);
+      score[e] = s;
+      choice[e] = s + (correction ? correction[e] : 0.f);
+    }
+  } else {
+    float m = -INFINITY;
+    for (int e = lane; e < E; e += 32) m = fmaxf(m, z[e]);
+    m = warp_max(m);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) {
+      const float x = expf(z[e] - m);
+      score[e] = x;
+      sum += x;
+    }
+    sum = warp_sum(sum);
+    for (int e = lane; e < E; e += 32) {
+      const float s = score[e] / sum;
+      score[e] = s;
+      choice[e] = s + (correction ? correction[e] : 0.f);
+    }
   }
   __syncwarp();
   if (groups > 1 && keep < groups) {
     const int per = E / groups;
     for (int g = 0; g < groups; ++g) {
-      float b = -INFINITY;
-      for (int e = lane; e < per; e += 32) b = fmaxf(b, choice[g * per + e]);
-      b = warp_max(b);
-      if (lane == 0) gbest[g] = b;
+      float b = -INFINITY, b2 = -INFINITY;           // the group's two largest choice scores
+      for (int e = lane; e < per; e += 32) {
+        const float c = choice[g * per + e];
+        b2 = fmaxf(b2, fminf(b, c));
+        b = fmaxf(b, c);
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, b, o), ob2 = __shfl_xor_sync(0xffffffffu, b2, o);
+        b2 = fmaxf(fmaxf(b2, ob2), fminf(b, ob));
+        b = fmaxf(b, ob);
+      }
+      if (lane == 0) gbest[g] = (group_best == 2 && per > 1) ? b + b2 : b;
     }
     __syncwarp();
     // the `keep` best groups stay; the others' choice scores become -inf (NaN marks a kept group in gbest)
@@ -523,7 +540,7 @@ softmax_group_topk_kernel(int32_t* __restrict__ ids, float* __restrict__ weights
     __syncwarp();
   }
   if (lane == 0) {
-    const float inv = 1.0f / (wsum + sum_floor);
+    const float inv = normalize ? weight_scale / (wsum + sum_floor) : weight_scale;
     for (int r = 0; r < top; ++r) weights[static_cast<int64_t>(tok) * top + r] *= inv;
   }
 }
@@ -712,19 +729,27 @@ int b200_cast_rows(void* out, const float* x, int64_t n, int dtype, void* stream
 
 int b200_softmax_group_topk(int32_t* ids, float* weights, const float* logits, const float* correction, float sum_floor,
                             int n_tok, int E, int top, int groups, int keep, void* stream) {
-  if (n_tok < 0 || E <= 0 || top <= 0 || top > E || groups < 1 || keep < 1 || keep > groups || E % groups)
-    return fail(B200_EINVAL, "b200_softmax_group_topk: bad sizes");
+  return b200_group_topk(ids, weights, logits, E, correction, 0, 1, 1, sum_floor, 1.0f, n_tok, E, top, groups, keep, stream);
+}
+
+int b200_group_topk(int32_t* ids, float* weights, const float* logits, int64_t logit_stride, const float* correction,
+                    int sigmoid_scores, int group_best, int normalize, float sum_floor, float weight_scale, int n_tok, int E,
+                    int top, int groups, int keep, void* stream) {
+  if (n_tok < 0 || E <= 0 || top <= 0 || top > E || groups < 1 || keep < 1 || keep > groups || E % groups ||
+      logit_stride < E || group_best < 1 || group_best > 2)
+    return fail(B200_EINVAL, "b200_group_topk: bad sizes");
   if (groups > 1 && keep < groups && static_cast<int64_t>(keep) * (E / groups) < top)
-    return fail(B200_EINVAL, "b200_softmax_group_topk: the kept groups hold fewer than `top` experts");
+    return fail(B200_EINVAL, "b200_group_topk: the kept groups hold fewer than `top` experts");
   if (n_tok == 0) return 0;
-  if (!ids || !weights || !logits) return fail(B200_EINVAL, "b200_softmax_group_topk: null pointer");
+  if (!ids || !weights || !logits) return fail(B200_EINVAL, "b200_group_topk: null pointer");
   const size_t smem = sizeof(float) * kRouteWarps * (2 * static_cast<size_t>(E) + groups);
-  if (smem > 200 * 1024) return fail(B200_ESHAPE, "b200_softmax_group_topk: %d experts are too many", E);
-  auto kern = softmax_group_topk_kernel;
+  if (smem > 200 * 1024) return fail(B200_ESHAPE, "b200_group_topk: %d experts are too many", E);
+  auto kern = group_topk_kernel;
   if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
   kern<<<(n_tok + kRouteWarps - 1) / kRouteWarps, kRouteWarps * 32, smem, static_cast<cudaStream_t>(stream)>>>(
-      ids, weights, logits, correction, sum_floor, n_tok, E, top, groups, keep);
-  return check_launch("b200_softmax_group_topk");
+      ids, weights, logits, logit_stride, correction, sigmoid_scores, group_best, normalize, sum_floor, weight_scale, n_tok, E,
+      top, groups, keep);
+  return check_launch("b200_group_topk");
 }
 
 int b200_gather_rows(void* xs, const void* h, const int64_t* src, int64_t n_rows, int top, int width, int dtype,

@@ -245,10 +245,10 @@ class GroupedSoftmaxMoE(nn.Module):
             return z[:, :z.shape[1] // 2]
         return mixer_ops.clamped_glu(z, self.limit, GLU_ALPHA)
 
-    def forward(self, h: torch.Tensor, x: torch.Tensor) -> torch.Tensor:
-        """``h``: the sublayer's input in the experts' dtype, ``x``: the same rows in fp32 (the residual)."""
+    def _experts(self, h: torch.Tensor, ids: torch.Tensor):
+        """The chosen experts' outputs: ``(ys [n * top, width] in expert order, where int64 [n * top])``; entry ``k`` of
+        token ``n`` is row ``where[n * top + k]``."""
         n, top, E = h.shape[0], self.top, self.E
-        ids, w = self._route(x)
         # rows in expert order; where each expert's rows start comes from the sorted ids themselves (a search, not a
         # count: no value ever travels to the host)
         # 16-bit keys: the radix sort takes two passes where 64-bit keys take eight (expert counts stay far below 2^15)
@@ -282,10 +282,16 @@ class GroupedSoftmaxMoE(nn.Module):
                     lo, hi = bounds[e], bounds[e + 1]
                     if hi > lo:
                         torch.mm(y[lo:hi], self.w_down[e].t(), out=ys[lo:hi])
+        return ys, where
+
+    def forward(self, h: torch.Tensor, x: torch.Tensor) -> torch.Tensor:
+        """``h``: the sublayer's input in the experts' dtype, ``x``: the same rows in fp32 (the residual)."""
+        ids, w = self._route(x)
+        ys, where = self._experts(h, ids)
         shared = None
         if self.ws_gu is not None:
             shared = F.linear(mixer_ops.clamped_glu(F.linear(h, self.ws_gu), self.shared_limit, GLU_ALPHA), self.ws_down)
-        return mixer_ops.weighted_expert_combine(ys, where, ids, w, x, shared, E)
+        return mixer_ops.weighted_expert_combine(ys, where, ids, w, x, shared, self.E)
 
 
 class FibiraxDecoderLayer(nn.Module):

@@ -513,19 +513,24 @@ def mixed_prompt_attention(out: torch.Tensor, q: torch.Tensor, k_pool: torch.Ten
 
 @_timed
 def causal_conv_silu(x: torch.Tensor, weight: torch.Tensor, tail: torch.Tensor, seqs: torch.Tensor,
-                     max_count: int) -> torch.Tensor:
-    """Short causal convolution per channel over each sequence's tokens, then SiLU.  ``x [n, C]`` (a column slice is
-    fine), ``weight [C, taps]`` (last column = the current token), ``tail`` fp32 ``[slots, taps - 1, C]`` carries each
-    live sequence's last inputs between steps and is updated."""
+                     max_count: int, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Short causal convolution per channel over each sequence's tokens (plus ``bias [C]``), then SiLU.  ``x [n, C]`` (a
+    column slice is fine), ``weight [C, taps]`` (last column = the current token), ``tail`` fp32 ``[slots, taps - 1, C]``
+    carries each live sequence's last inputs between steps and is updated."""
     _need_cuda(x, weight, tail, seqs)
     C, taps = weight.shape
     if x.shape[1] != C or tail.dtype != torch.float32 or tuple(tail.shape[1:]) != (taps - 1, C) or not tail.is_contiguous():
         raise ValueError("x [n, C], weight [C, taps], tail fp32 [slots, taps - 1, C]")
     if seqs.dtype != torch.int32 or seqs.dim() != 2 or seqs.shape[1] != 4 or not seqs.is_contiguous():
         raise ValueError("seqs must be contiguous int32 [n_seqs, 4]")
+    if bias is not None and (bias.numel() != C or bias.dtype != x.dtype or not bias.is_contiguous()):
+        raise ValueError("bias is contiguous [C] in the activations' dtype")
+    if weight.dtype != x.dtype or not weight.is_contiguous():
+        raise ValueError("weight is contiguous [C, taps] in the activations' dtype")
     out = torch.empty((x.shape[0], C), dtype=x.dtype, device=x.device)
-    rc = _lib_().b200_causal_conv_silu(out.data_ptr(), C, x.data_ptr(), _rows2(x), weight.data_ptr(), tail.data_ptr(),
-                                       seqs.data_ptr(), seqs.shape[0], int(max_count), C, taps, DTYPE_ID[x.dtype], _stream())
+    rc = _lib_().b200_causal_conv_silu_ext(out.data_ptr(), C, x.data_ptr(), _rows2(x), weight.data_ptr(), _ptr(bias),
+                                           tail.data_ptr(), seqs.data_ptr(), seqs.shape[0], int(max_count), C, taps,
+                                           DTYPE_ID[x.dtype], _stream())
     _lib.check_mixers(rc, "b200_causal_conv_silu")
     return out
 
@@ -813,11 +818,12 @@ def token_shift(x: torch.Tensor, mu: torch.Tensor, state: torch.Tensor, seqs: to
 @_timed
 def latent_rotary_append(q_rot: torch.Tensor, q_out: torch.Tensor, dkv: torch.Tensor, c_norm: torch.Tensor, eps: float,
                          freqs: Optional[torch.Tensor], gain: float, pool: torch.Tensor, slot_mapping: torch.Tensor,
-                         tok_pos: torch.Tensor) -> None:
+                         tok_pos: torch.Tensor, interleaved: bool = True) -> None:
     """``dkv [n, rank + dr]``: its first ``rank = len(c_norm)`` columns RMS-normed with ``c_norm`` and its last ``dr``
     turned by the position go to one row of the one-head ``pool [blocks, 1, bs, rank + dr]``; ``q_out[n, h, :] =
     turn(q_rot[n, h, :])`` for 3-D views ``[n, H, dr]`` with contiguous last dimensions that do not overlap.  Pairs
-    ``(2i, 2i + 1)``, ``i < len(freqs)``, are turned by ``pos * freqs[i]`` with cos and sin times ``gain``."""
+    ``(2i, 2i + 1)`` (``interleaved``) or ``(i, i + len(freqs))``, ``i < len(freqs)``, are turned by ``pos * freqs[i]`` with
+    cos and sin times ``gain``."""
     _need_cuda(q_rot, q_out, dkv, c_norm, pool, slot_mapping, tok_pos)
     n, H, dr = q_rot.shape
     rank = c_norm.numel()
@@ -836,11 +842,11 @@ def latent_rotary_append(q_rot: torch.Tensor, q_out: torch.Tensor, dkv: torch.Te
         if freqs.dtype != torch.float64 or not freqs.is_contiguous() or not freqs.is_cuda:
             raise ValueError("freqs is a contiguous float64 tensor on the device")
         rot_dims = 2 * freqs.numel()
-    rc = _lib_().b200_latent_rotary_append(q_rot.data_ptr(), q_rot.stride(0), q_rot.stride(1), q_out.data_ptr(),
-                                           q_out.stride(0), q_out.stride(1), dkv.data_ptr(), _rows2(dkv), c_norm.data_ptr(),
-                                           float(eps), _ptr(freqs), float(gain), rot_dims, pool.data_ptr(),
-                                           slot_mapping.data_ptr(), tok_pos.data_ptr(), n, H, dr, rank, DTYPE_ID[T],
-                                           _stream())
+    rc = _lib_().b200_latent_rotary_append_ext(q_rot.data_ptr(), q_rot.stride(0), q_rot.stride(1), q_out.data_ptr(),
+                                               q_out.stride(0), q_out.stride(1), dkv.data_ptr(), _rows2(dkv),
+                                               c_norm.data_ptr(), float(eps), _ptr(freqs), float(gain), rot_dims,
+                                               int(interleaved), pool.data_ptr(), slot_mapping.data_ptr(),
+                                               tok_pos.data_ptr(), n, H, dr, rank, DTYPE_ID[T], _stream())
     _lib.check_mixers(rc, "b200_latent_rotary_append")
 
 
@@ -920,16 +926,258 @@ def gated_table_rows(z: torch.Tensor, table: torch.Tensor, col0: int, tokens: to
 
 @_timed
 def router_logits(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """fp32 ``x [n, width] @ w [E, width].T + bias``: a router's logits, every sum in an order fixed by the width (a
-    token's choice of experts does not depend on the rest of the step)."""
+    """``x [n, width] @ w [E, width].T + bias`` in fp32: a router's logits, every sum in an order fixed by the width (a
+    token's choice of experts does not depend on the rest of the step).  ``x`` may be of any storage dtype."""
     _need_cuda(x, w)
-    if x.dtype != torch.float32 or w.dtype != torch.float32 or x.dim() != 2 or w.dim() != 2 or x.shape[1] != w.shape[1] \
+    if w.dtype != torch.float32 or x.dim() != 2 or w.dim() != 2 or x.shape[1] != w.shape[1] \
             or not x.is_contiguous() or not w.is_contiguous():
-        raise ValueError("x [n, width] and w [E, width] are contiguous fp32")
+        raise ValueError("x [n, width] is contiguous and w [E, width] contiguous fp32")
     if bias is not None and (bias.dtype != torch.float32 or bias.numel() != w.shape[0] or not bias.is_contiguous()):
         raise ValueError("bias is contiguous fp32 [E]")
     out = torch.empty((x.shape[0], w.shape[0]), dtype=torch.float32, device=x.device)
-    rc = _lib_().b200_router_logits(out.data_ptr(), x.data_ptr(), w.data_ptr(), _ptr(bias), x.shape[0], w.shape[0],
-                                    x.shape[1], _stream())
+    rc = _lib_().b200_router_logits_ext(out.data_ptr(), x.data_ptr(), w.data_ptr(), _ptr(bias), x.shape[0], w.shape[0],
+                                        x.shape[1], DTYPE_ID[x.dtype], _stream())
     _lib.check_mixers(rc, "b200_router_logits")
+    return out
+
+
+# ---- recurrences decayed by one number per token and head, dynamic tanh norms (csrc/b200_recurrent_ops.cu) ------------
+@_timed
+def sigmoid_group_topk(logits: torch.Tensor, correction: Optional[torch.Tensor], n_experts: int, top: int, groups: int = 1,
+                       keep: int = 1, scale: float = 1.0):
+    """fp32 logits rows (their first ``n_experts`` columns) -> ``(ids int32 [n, top], weights fp32 [n, top])``: sigmoid
+    scores, the choice by score + ``correction`` inside the ``keep`` of ``groups`` expert groups whose two largest choice
+    scores have the largest sum, weights = ``scale`` times the chosen scores."""
+    _need_cuda(logits)
+    n, E = logits.shape[0], int(n_experts)
+    if logits.dtype != torch.float32 or logits.dim() != 2 or logits.shape[1] < E:
+        raise ValueError("router logits are fp32 [n, >= n_experts]")
+    if correction is not None and (correction.dtype != torch.float32 or correction.numel() != E
+                                   or not correction.is_contiguous()):
+        raise ValueError("correction is contiguous fp32 [n_experts]")
+    ids = torch.empty((n, top), dtype=torch.int32, device=logits.device)
+    w = torch.empty((n, top), dtype=torch.float32, device=logits.device)
+    rc = _lib_().b200_group_topk(ids.data_ptr(), w.data_ptr(), logits.data_ptr(), _rows2(logits), _ptr(correction), 1, 2, 0,
+                                 0.0, float(scale), n, E, int(top), int(groups), int(keep), _stream())
+    _lib.check_mixers(rc, "b200_group_topk")
+    return ids, w
+
+
+def _check_dyn_tanh(x: torch.Tensor, w: Optional[torch.Tensor], b: Optional[torch.Tensor], T: torch.dtype) -> None:
+    if x.dtype != torch.float32 or not x.is_contiguous() or x.dim() != 2:
+        raise ValueError("the residual stream is a contiguous fp32 [rows, width] tensor")
+    for t in (w, b):
+        if t is not None and (t.dtype != T or t.numel() != x.shape[1] or not t.is_contiguous()):
+            raise ValueError("norm weight and bias are contiguous [width] in one dtype")
+
+
+@_timed
+def residual_dyn_tanh(x: torch.Tensor, y: Optional[torch.Tensor], norm=None) -> Optional[torch.Tensor]:
+    """In place ``x += y`` on the fp32 residual (``y`` fp32 or of the norm's dtype; None: no update); with ``norm = (weight,
+    bias, alpha)`` returns ``tanh(alpha x) * weight + bias`` of the new residual in the weight's dtype."""
+    _need_cuda(x)
+    w, b, alpha = norm if norm is not None else (None, None, 0.0)
+    T = w.dtype if w is not None else (y.dtype if y is not None else torch.float32)
+    _check_dyn_tanh(x, w, b, T)
+    if y is not None and (y.shape != x.shape or y.dtype not in (T, torch.float32)):
+        raise ValueError("y has the residual's shape and is fp32 or of the norm's dtype")
+    out = torch.empty(x.shape, dtype=T, device=x.device) if w is not None else None
+    rc = _lib_().b200_residual_dyn_tanh(x.data_ptr(), _ptr(y), _rows2(y) if y is not None else 0,
+                                        int(y is not None and y.dtype == torch.float32 and T != torch.float32), _ptr(w),
+                                        _ptr(b), float(alpha), _ptr(out), x.shape[0], x.shape[1], DTYPE_ID[T], _stream())
+    _lib.check_mixers(rc, "b200_residual_dyn_tanh")
+    return out
+
+
+@_timed
+def expert_combine_dyn_tanh(x: torch.Tensor, ys: torch.Tensor, where: torch.Tensor, weights: torch.Tensor,
+                            shared: Optional[torch.Tensor], shared_gate: Optional[torch.Tensor], norm=None
+                            ) -> Optional[torch.Tensor]:
+    """In place ``x[n] += sum_k weights[n, k] * ys[where[n*top + k]] + sigmoid(shared_gate[n]) * shared[n]`` on the fp32
+    residual; ``shared_gate`` is a 1-D fp32 view of logits (any stride, None: factor 1).  ``norm`` as in
+    ``residual_dyn_tanh``."""
+    _need_cuda(x, ys, where, weights)
+    w, b, alpha = norm if norm is not None else (None, None, 0.0)
+    T = ys.dtype
+    _check_dyn_tanh(x, w, b, T)
+    n, top = weights.shape
+    if not ys.is_contiguous() or ys.shape[1] != x.shape[1] or where.dtype != torch.int64 or where.numel() != n * top:
+        raise ValueError("ys contiguous [rows, width], where int64 [n * top]")
+    if weights.dtype != torch.float32 or not weights.is_contiguous() or n != x.shape[0]:
+        raise ValueError("weights contiguous fp32 [n, top]")
+    if shared is not None and (shared.shape != x.shape or shared.dtype != T or not shared.is_contiguous()):
+        raise ValueError("shared rows are contiguous [n, width] in the experts' dtype")
+    if shared_gate is not None and (shared_gate.dtype != torch.float32 or shared_gate.dim() != 1 or shared_gate.numel() != n):
+        raise ValueError("shared_gate is fp32 [n]")
+    out = torch.empty(x.shape, dtype=T, device=x.device) if w is not None else None
+    rc = _lib_().b200_expert_combine_dyn_tanh(x.data_ptr(), ys.data_ptr(), where.data_ptr(), weights.data_ptr(), top,
+                                              _ptr(shared), _ptr(shared_gate),
+                                              shared_gate.stride(0) if shared_gate is not None else 0, _ptr(w), _ptr(b),
+                                              float(alpha), _ptr(out), n, x.shape[1], DTYPE_ID[T], _stream())
+    _lib.check_mixers(rc, "b200_expert_combine_dyn_tanh")
+    return out
+
+
+@_timed
+def silu_glu(gu: torch.Tensor) -> torch.Tensor:
+    """``silu(g) * u`` of contiguous rows ``g | u``."""
+    _need_cuda(gu)
+    if not gu.is_contiguous() or gu.dim() != 2 or gu.shape[1] % 2:
+        raise ValueError("gu must be contiguous [rows, 2*ff]")
+    ff = gu.shape[1] // 2
+    y = torch.empty((gu.shape[0], ff), dtype=gu.dtype, device=gu.device)
+    rc = _lib_().b200_silu_glu(y.data_ptr(), gu.data_ptr(), gu.shape[0], ff, DTYPE_ID[gu.dtype], _stream())
+    _lib.check_mixers(rc, "b200_silu_glu")
+    return y
+
+
+def _f32_heads(*tensors: torch.Tensor, H: int) -> None:
+    for t in tensors:
+        if t is not None and (t.dtype != torch.float32 or t.numel() != H or not t.is_contiguous()):
+            raise ValueError("per-head constants are contiguous fp32 [H]")
+
+
+@_timed
+def capped_gates(zi: torch.Tensor, zf: torch.Tensor, bias_i: torch.Tensor, bias_f: torch.Tensor, cap: float,
+                 m_state: torch.Tensor, seqs: torch.Tensor):
+    """Exponential gates with a soft cap and a running maximum: ``(decay, coef, m)``, fp32 ``[n, H]`` each (see
+    ``b200_capped_gates``).  ``zi / zf [n, H]`` are column slices of one projection; ``m_state`` fp32 ``[slots, H]`` carries
+    the maximum and is updated."""
+    _need_cuda(zi, zf, m_state, seqs)
+    _check_seqs(seqs)
+    n, H = zi.shape
+    _f32_heads(bias_i, bias_f, H=H)
+    if zf.shape != zi.shape or zf.dtype != zi.dtype or (n > 1 and zf.stride(0) != zi.stride(0)):
+        raise ValueError("zi and zf are [n, H] slices with one row stride")
+    if m_state.dtype != torch.float32 or m_state.shape[1:] != (H,) or not m_state.is_contiguous():
+        raise ValueError("m_state is contiguous fp32 [slots, H]")
+    decay, coef, m = torch.empty((3, n, H), dtype=torch.float32, device=zi.device).unbind(0)
+    rc = _lib_().b200_capped_gates(decay.data_ptr(), coef.data_ptr(), m.data_ptr(), zi.data_ptr(), zf.data_ptr(), _rows2(zi),
+                                   bias_i.data_ptr(), bias_f.data_ptr(), float(cap), m_state.data_ptr(), seqs.data_ptr(),
+                                   seqs.shape[0], H, DTYPE_ID[zi.dtype], _stream())
+    _lib.check_mixers(rc, "b200_capped_gates")
+    return decay, coef, m
+
+
+@_timed
+def step_sizes(z: torch.Tensor, bias: torch.Tensor, a_log: torch.Tensor):
+    """``dt = softplus(z + bias)``, ``decay = exp(-exp(a_log) dt)``: ``(decay, dt)``, fp32 ``[n, H]``."""
+    _need_cuda(z)
+    n, H = z.shape
+    _f32_heads(bias, a_log, H=H)
+    decay, coef = torch.empty((2, n, H), dtype=torch.float32, device=z.device).unbind(0)
+    rc = _lib_().b200_step_sizes(decay.data_ptr(), coef.data_ptr(), z.data_ptr(), _rows2(z), bias.data_ptr(), a_log.data_ptr(),
+                                 n, H, DTYPE_ID[z.dtype], _stream())
+    _lib.check_mixers(rc, "b200_step_sizes")
+    return decay, coef
+
+
+def _check_decay_inputs(q, k, v, state, nstate, seqs, G: int):
+    _need_cuda(q, k, v, state, seqs)
+    _check_seqs(seqs)
+    n = q.shape[0]
+    _, H, dk, dv = state.shape
+    if H % G or q.shape[1] != G * dk or k.shape != q.shape or v.shape != (n, H * dv):
+        raise ValueError("projections do not match the state's shape")
+    if k.dtype != q.dtype or v.dtype != q.dtype:
+        raise TypeError("q, k and v share one dtype")
+    if state.dtype != torch.float32 or not state.is_contiguous():
+        raise TypeError("the recurrent state is contiguous fp32")
+    if nstate is not None and (nstate.dtype != torch.float32 or nstate.shape[1:] != (H, dk) or not nstate.is_contiguous()):
+        raise ValueError("nstate is contiguous fp32 [slots, H, dk]")
+    return n, H, dk, dv
+
+
+@_timed
+def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, coef: torch.Tensor,
+               state: torch.Tensor, seqs: torch.Tensor, G: int, q_scale: float = 1.0, skip: Optional[torch.Tensor] = None,
+               nstate: Optional[torch.Tensor] = None):
+    """``S <- decay S + coef k v^T``, ``o = S^T (q_scale q) + skip v`` over each sequence's tokens, and with ``nstate`` the
+    vector recurrence ``n <- decay n + coef k`` and ``n . (q_scale q)``.  ``q / k [n, G*dk]``, ``v [n, H*dv]``, ``decay /
+    coef`` fp32 ``[n, H]``, ``state`` fp32 ``[slots, H, dk, dv]``.  Returns ``(o fp32 [n, H, dv], nq fp32 [n, H] or None)``."""
+    n, H, dk, dv = _check_decay_inputs(q, k, v, state, nstate, seqs, G)
+    _f32_heads(skip, H=H)
+    for t in (decay, coef):
+        if t.dtype != torch.float32 or tuple(t.shape) != (n, H) or not t.is_contiguous():
+            raise ValueError("decay and coef are contiguous fp32 [n, H]")
+    o = torch.empty((n, H, dv), dtype=torch.float32, device=q.device)
+    nq = torch.empty((n, H), dtype=torch.float32, device=q.device) if nstate is not None else None
+    rc = _lib_().b200_decay_scan(o.data_ptr(), _ptr(nq), q.data_ptr(), _rows2(q), k.data_ptr(), _rows2(k), v.data_ptr(),
+                                 _rows2(v), decay.data_ptr(), coef.data_ptr(), _ptr(skip), float(q_scale), state.data_ptr(),
+                                 _ptr(nstate), seqs.data_ptr(), seqs.shape[0], H, G, dk, dv, DTYPE_ID[q.dtype], _stream())
+    _lib.check_mixers(rc, "b200_decay_scan")
+    return o, nq
+
+
+@_timed
+def decay_step(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, gates, state: torch.Tensor, seqs: torch.Tensor, G: int,
+               q_scale: float = 1.0, skip: Optional[torch.Tensor] = None, nstate: Optional[torch.Tensor] = None,
+               m_state: Optional[torch.Tensor] = None):
+    """``decay_scan`` for steps of one token per sequence, the gates formed on the way.  ``gates``: ``("capped", zi, zf,
+    bias_i, bias_f, cap)`` with ``m_state`` (only read), or ``("step", z, bias, a_log)``.  Returns ``(o, nq, m)``."""
+    n, H, dk, dv = _check_decay_inputs(q, k, v, state, nstate, seqs, G)
+    if seqs.shape[0] != n:
+        raise ValueError("decay_step serves one token per sequence")
+    _f32_heads(skip, H=H)
+    capped = gates[0] == "capped"
+    if capped:
+        _, za, zb, p0, p1, cap = gates
+        if zb.shape != za.shape or (n > 1 and zb.stride(0) != za.stride(0)) or m_state is None \
+                or m_state.dtype != torch.float32 or m_state.shape[1:] != (H,) or not m_state.is_contiguous():
+            raise ValueError("zi and zf are [n, H] slices with one row stride; m_state is fp32 [slots, H]")
+    else:
+        (_, za, p0, p1), zb, cap = gates, None, 1.0
+    if tuple(za.shape) != (n, H) or za.dtype != q.dtype:
+        raise ValueError("gate logits are [n, H] in the activations' dtype")
+    _f32_heads(p0, p1, H=H)
+    o = torch.empty((n, H, dv), dtype=torch.float32, device=q.device)
+    nq = torch.empty((n, H), dtype=torch.float32, device=q.device) if nstate is not None else None
+    m = torch.empty((n, H), dtype=torch.float32, device=q.device) if capped else None
+    rc = _lib_().b200_decay_step(o.data_ptr(), _ptr(nq), _ptr(m), q.data_ptr(), _rows2(q), k.data_ptr(), _rows2(k),
+                                 v.data_ptr(), _rows2(v), 0 if capped else 1, za.data_ptr(), _ptr(zb), _rows2(za),
+                                 p0.data_ptr(), p1.data_ptr(), float(cap), _ptr(skip), float(q_scale), state.data_ptr(),
+                                 _ptr(nstate), _ptr(m_state), seqs.data_ptr(), n, H, G, dk, dv, DTYPE_ID[q.dtype], _stream())
+    _lib.check_mixers(rc, "b200_decay_step")
+    return o, nq, m
+
+
+@_timed
+def normalized_head_out(o: torch.Tensor, nq: torch.Tensor, m: torch.Tensor, floor: float, weight: torch.Tensor,
+                        gate: torch.Tensor, eps: float, m_state: Optional[torch.Tensor] = None,
+                        seqs: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """fp32 ``o [n, H, dv]`` over ``max(|nq|, exp(-m)) + floor`` per head, made unit-RMS per head, times ``weight [H*dv]``,
+    times ``sigmoid(gate [n, H*dv])``: ``[n, H*dv]`` in the weight's dtype.  With ``m_state`` (steps of one token per
+    sequence) the running maxima ``m`` are stored at the sequences' slots."""
+    _need_cuda(o, nq, m, weight, gate)
+    n, H, dv = o.shape
+    if any(t.dtype != torch.float32 or not t.is_contiguous() for t in (o, nq, m)) or nq.shape != (n, H) or m.shape != (n, H):
+        raise ValueError("o [n, H, dv], nq and m [n, H] are contiguous fp32")
+    if weight.numel() != H * dv or not weight.is_contiguous() or tuple(gate.shape) != (n, H * dv) or gate.dtype != weight.dtype:
+        raise ValueError("weight [H*dv] and gate [n, H*dv] share one dtype")
+    if m_state is not None:
+        _check_seqs(seqs)
+        if seqs.shape[0] != n or m_state.dtype != torch.float32 or m_state.shape[1:] != (H,) or not m_state.is_contiguous():
+            raise ValueError("m_state is contiguous fp32 [slots, H], one sequence per row")
+    out = torch.empty((n, H * dv), dtype=weight.dtype, device=o.device)
+    rc = _lib_().b200_normalized_head_out(out.data_ptr(), H * dv, o.data_ptr(), nq.data_ptr(), m.data_ptr(), float(floor),
+                                          weight.data_ptr(), gate.data_ptr(), _rows2(gate), float(eps), _ptr(m_state),
+                                          _ptr(seqs), n, H, dv, DTYPE_ID[weight.dtype], _stream())
+    _lib.check_mixers(rc, "b200_normalized_head_out")
+    return out
+
+
+@_timed
+def gated_part_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, eps: float, parts: int) -> torch.Tensor:
+    """``y * silu(z)`` with each of ``parts`` equal parts of the row divided by its own RMS, times ``weight``: fp32 ``y [n,
+    inner]``, ``z`` and the result in the weight's dtype."""
+    _need_cuda(y, z, weight)
+    n, inner = z.shape
+    if y.dtype != torch.float32 or not y.is_contiguous() or y.numel() != n * inner:
+        raise ValueError("y is contiguous fp32 [n, inner]")
+    if weight.numel() != inner or not weight.is_contiguous() or z.dtype != weight.dtype or inner % parts:
+        raise ValueError("weight is [inner] in z's dtype and the parts divide the row")
+    out = torch.empty((n, inner), dtype=weight.dtype, device=y.device)
+    rc = _lib_().b200_gated_part_norm(out.data_ptr(), y.data_ptr(), z.data_ptr(), _rows2(z), weight.data_ptr(), float(eps), n,
+                                      inner, int(parts), DTYPE_ID[weight.dtype], _stream())
+    _lib.check_mixers(rc, "b200_gated_part_norm")
     return out

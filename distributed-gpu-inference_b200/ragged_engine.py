@@ -245,7 +245,9 @@ class RaggedStepEngine:
             return last.get_logits(rows).to(torch.float32)
         if self._head_f32 is None:   # fp32 accumulation AND fp32 output of the storage-dtype operands
             self._head_f32 = last.lm_head.weight.detach().to(torch.float32)
-        return F.linear(rows.to(torch.float32), self._head_f32)
+        logits = F.linear(rows.to(torch.float32), self._head_f32)
+        scale = getattr(last.lm_head, "logit_scale", 1.0)      # a head that scales its logits does so in its own forward
+        return logits if scale == 1.0 else logits * scale
 
     # ---- scheduler -----------------------------------------------------------------------------------------------
     @torch.no_grad()

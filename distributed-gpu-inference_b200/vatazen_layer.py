@@ -136,8 +136,9 @@ class LatentRotaryAttention(nn.Module):
 
     HEADS_AS_ROWS_FROM = 16    # heads from which a step of single tokens puts heads on the rows of the attention's tiles
 
-    def __init__(self, spec: Dict[str, Any], t: Dict[str, torch.Tensor], eps: float, device, dtype):
+    def __init__(self, spec: Dict[str, Any], t: Dict[str, torch.Tensor], eps: float, device, dtype, interleaved: bool = True):
         super().__init__()
+        self.interleaved = interleaved      # rotary pairs (2i, 2i + 1); False: (i, i + half)
         self.H, self.dn, self.dr = int(spec["heads"]), int(spec["dim"]), int(spec["rot_dim"])
         self.dv, self.rank = int(spec["vdim"]), int(spec["kv_rank"])
         self.scale, self.eps = float(spec["scale"]), eps
@@ -166,7 +167,7 @@ class LatentRotaryAttention(nn.Module):
         q = proj[:, :H * (dn + dr)].unflatten(1, (H, dn + dr))
         q_lat = torch.empty((n, H, r + dr), dtype=h.dtype, device=h.device)       # [W_uk^T q_plain | turned q part]
         mixer_ops.latent_rotary_append(q[:, :, dn:], q_lat[:, :, r:], proj[:, c[1]:c[1] + r + dr], self.c_norm, self.eps,
-                                       self.freqs, self.gain, cache.k_pool, st.slot_mapping, st.tok_pos)
+                                       self.freqs, self.gain, cache.k_pool, st.slot_mapping, st.tok_pos, self.interleaved)
         torch.bmm(q[:, :, :dn].transpose(0, 1), self.w_uk, out=q_lat[:, :, :r].transpose(0, 1))
         o_lat = torch.empty((H, n, r), dtype=h.dtype, device=h.device)
         if self.tensor_cores:

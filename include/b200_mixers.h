@@ -348,6 +348,92 @@ int b200_gated_table_rows(void* out, const void* z, int64_t z_stride, const void
 int b200_router_logits(float* logits, const float* x, const float* w, const float* bias, int64_t n_tok, int E, int width,
                        void* stream);
 
+/* b200_causal_conv_silu with a bias per channel (T [C], may be NULL) added before the SiLU.  taps <= 16. */
+int b200_causal_conv_silu_ext(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* w, const void* bias,
+                              float* tail, const int32_t* seqs, int n_seqs, int max_count, int C, int taps, int dtype,
+                              void* stream);
+
+/* b200_latent_rotary_append with the pair layout as an argument: interleaved != 0: pairs (2i, 2i + 1); 0: pairs
+ * (i, i + rot_dims / 2). */
+int b200_latent_rotary_append_ext(const void* q_rot, int64_t q_tok_stride, int64_t q_head_stride, void* q_out,
+                                  int64_t qo_tok_stride, int64_t qo_head_stride, const void* dkv, int64_t dkv_stride,
+                                  const void* c_norm, float eps, const double* freqs, float gain, int rot_dims,
+                                  int interleaved, void* pool, const int64_t* slot_mapping, const int32_t* tok_pos, int n_tok,
+                                  int H, int rot_width, int rank, int dtype, void* stream);
+
+/* b200_router_logits with x in any storage type (dtype; w, bias and the sums stay fp32). */
+int b200_router_logits_ext(float* logits, const void* x, const float* w, const float* bias, int64_t n_tok, int E, int width,
+                           int dtype, void* stream);
+
+/* Routing over E outputs (the first E of every logits row; rows are logit_stride apart): scores s = softmax over the E logits
+ * or, with sigmoid_scores, the logits' sigmoids; choice scores c = s + correction (NULL: c = s); a group's score is its largest
+ * c or, with group_best = 2, the sum of its two largest; groups, keep and top as in b200_softmax_group_topk.  weights =
+ * weight_scale * s, divided by (the sum of the chosen s + sum_floor) with normalize. */
+int b200_group_topk(int32_t* ids, float* weights, const float* logits, int64_t logit_stride, const float* correction,
+                    int sigmoid_scores, int group_best, int normalize, float sum_floor, float weight_scale, int n_tok, int E,
+                    int top, int groups, int keep, void* stream);
+
+/* ---- pieces for designs with recurrences decayed by one number per token and head, and dynamic tanh norms ---------- */
+
+/* x[r] += y[r] in fp32, in place (y may be NULL; T, or fp32 with y_is_f32); out[r] = tanh(alpha x[r]) * w + b in T
+ * (out may be NULL).  x fp32 [rows, width] contiguous; w, b T [width]. */
+int b200_residual_dyn_tanh(float* x, const void* y, int64_t y_stride, int y_is_f32, const void* w, const void* b, float alpha,
+                           void* out, int64_t rows, int width, int dtype, void* stream);
+
+/* x[n] += sum over k (ascending) of weights[n][k] * ys[where[n * top + k]] + sigmoid(shared_gate[n * gate_stride]) *
+ * shared_rows[n] in fp32, in place (shared_rows may be NULL; shared_gate NULL: factor 1); out as in b200_residual_dyn_tanh. */
+int b200_expert_combine_dyn_tanh(float* x, const void* ys, const int64_t* where, const float* weights, int top,
+                                 const void* shared_rows, const float* shared_gate, int64_t gate_stride, const void* w,
+                                 const void* b, float alpha, void* out, int64_t n_tok, int width, int dtype, void* stream);
+
+/* y = silu(g) * u; gu rows = g | u, contiguous [rows, 2 * ff]. */
+int b200_silu_glu(void* y, const void* gu, int64_t rows, int ff, int dtype, void* stream);
+
+/* Capped exponential gates of a step's portions (SeqSpan rows): with sc(z) = cap * tanh(z / cap), i = sc(zi + bias_i),
+ * f = log sigmoid(sc(zf + bias_f)) and the running maximum m_t = max(f + m_(t-1), i):
+ *   decay = exp(f + m_(t-1) - m_t),  coef = exp(i - m_t),  m_seq = m_t          fp32 [n_tok, H]
+ * zi, zf: T rows [n_tok, H] with row stride z_stride; biases fp32 [H]; m_state fp32 [slots, H] carries m (0 when the sequence
+ * is fresh) and is updated. */
+int b200_capped_gates(float* decay, float* coef, float* m_seq, const void* zi, const void* zf, int64_t z_stride,
+                      const float* bias_i, const float* bias_f, float cap, float* m_state, const int32_t* seqs, int n_seqs,
+                      int H, int dtype, void* stream);
+
+/* Step sizes: coef = dt = softplus(z + bias), decay = exp(-exp(a_log) * dt); z T rows [n_tok, H]; bias, a_log fp32 [H]. */
+int b200_step_sizes(float* decay, float* coef, const void* z, int64_t z_stride, const float* bias, const float* a_log,
+                    int64_t n_tok, int H, int dtype, void* stream);
+
+/* Decayed outer-product state per (sequence, head) over the sequence's tokens of this step, in order (SeqSpan rows):
+ *   S <- decay[t][h] S + coef[t][h] k_t v_t^T;   o_t = S^T (q_scale q_t) + skip[h] v_t              (skip may be NULL)
+ *   n <- decay[t][h] n + coef[t][h] k_t;         nq_t = n . (q_scale q_t)                           (nstate NULL: no n)
+ * q, k: T rows of G*dk (head h reads head h / (H / G)), v: T rows of H*dv, each with its row stride; decay, coef fp32
+ * [n_tok, H]; skip fp32 [H]; state fp32 [slots, H, dk, dv] and nstate fp32 [slots, H, dk], read unless the sequence is fresh
+ * and written back; o fp32 [n_tok, H, dv], nq fp32 [n_tok, H].  dk <= 512. */
+int b200_decay_scan(float* o, float* nq, const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v,
+                    int64_t v_stride, const float* decay, const float* coef, const float* skip, float q_scale, float* state,
+                    float* nstate, const int32_t* seqs, int n_seqs, int H, int G, int dk, int dv, int dtype, void* stream);
+
+/* The same for steps whose sequences bring ONE token each (row n = sequence n), decay and coef formed on the way:
+ * gate_kind 0: b200_capped_gates with za = zi, zb = zf, p0 = bias_i, p1 = bias_f; m_seq [n_tok, H] receives the new running
+ * maximum, m_state is only read (b200_normalized_head_out stores it); gate_kind 1: b200_step_sizes with za = z, p0 = bias,
+ * p1 = a_log (zb, m_seq, m_state NULL). */
+int b200_decay_step(float* o, float* nq, float* m_seq, const void* q, int64_t q_stride, const void* k, int64_t k_stride,
+                    const void* v, int64_t v_stride, int gate_kind, const void* za, const void* zb, int64_t z_stride,
+                    const float* p0, const float* p1, float cap, const float* skip, float q_scale, float* state,
+                    float* nstate, const float* m_state, const int32_t* seqs, int n_seqs, int H, int G, int dk, int dv,
+                    int dtype, void* stream);
+
+/* y = o[n][h] / (max(|nq[n][h]|, exp(-m_seq[n][h])) + floor);  out[n, h*dv + i] = y_i * rsqrt(mean_i y^2 + eps) * w[h*dv + i] *
+ * sigmoid(gate[n, h*dv + i]).  w T [H*dv], gate T rows.  m_state (may be NULL; steps of one token per sequence): receives
+ * m_seq at the sequences' slots. */
+int b200_normalized_head_out(void* out, int64_t out_stride, const float* o, const float* nq, const float* m_seq, float floor_,
+                             const void* w, const void* gate, int64_t gate_stride, float eps, float* m_state,
+                             const int32_t* seqs, int64_t n_tok, int H, int dv, int dtype, void* stream);
+
+/* v = y * silu(z);  out = v * rsqrt(mean over its part of v^2 + eps) * w, the row of `inner` cut into `parts` equal parts.
+ * y fp32 [n_tok, inner] contiguous, z T rows, w T [inner], out T [n_tok, inner]. */
+int b200_gated_part_norm(void* out, const float* y, const void* z, int64_t z_stride, const void* w, float eps, int64_t n_tok,
+                         int inner, int parts, int dtype, void* stream);
+
 #ifdef __cplusplus
 }
 #endif
