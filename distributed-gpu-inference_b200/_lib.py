@@ -214,7 +214,7 @@ MIXER_SIGNATURES = {
     "b200_router_logits": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_int, c_int, c_void_p]),
     "b200_gated_table_rows": (
         c_int, [c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_int, c_void_p, c_int64, c_int, c_int, c_void_p]),
-    # one decay per token and head, dynamic tanh norms, sigmoid group routing (csrc/b200_recurrent_ops.cu)
+    # one decay per token and head, dynamic tanh norms, sigmoid group routing (csrc/b200_recurrent_ops.cu, csrc/b200_chunk_scan.cu)
     "b200_causal_conv_silu_ext": (
         c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int,
                 c_int, c_int, c_int, c_void_p]),
@@ -241,6 +241,11 @@ MIXER_SIGNATURES = {
     "b200_step_sizes": (
         c_int, [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int, c_int, c_void_p]),
     "b200_decay_scan": (
+        c_int, [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
+                c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
+                c_int, c_int, c_void_p]),
+    "b200_decay_chunk_scan_supported": (c_int, [c_int, c_int, c_int]),
+    "b200_decay_chunk_scan": (
         c_int, [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
                 c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int,
                 c_int, c_int, c_void_p]),
@@ -309,7 +314,7 @@ def _build_mixers() -> None:
         fcntl.flock(lock, fcntl.LOCK_EX)
         if os.path.exists(MIXER_LIB_PATH):
             return
-        proc = subprocess.run(["make", "-j5", "-C", csrc, "mixers"], stdout=subprocess.PIPE, stderr=subprocess.STDOUT)
+        proc = subprocess.run(["make", "-j6", "-C", csrc, "mixers"], stdout=subprocess.PIPE, stderr=subprocess.STDOUT)
         if proc.returncode != 0 or not os.path.exists(MIXER_LIB_PATH):
             raise B200LibraryError("building libb200_mixers.so failed:\n" + proc.stdout.decode(errors="replace")[-4000:])
 

@@ -228,9 +228,9 @@ __device__ __forceinline__ void gate_logs(const DecayGates& G, int64_t n, int h,
 }
 
 template <typename T>
-__device__ __forceinline__ void step_size(const DecayGates& G, int64_t n, int h, float& d, float& c) {
+__device__ __forceinline__ void step_size(const DecayGates& G, int64_t n, int h, float& log_d, float& c) {
   c = softplus1(Cvt<T>::to_f32(static_cast<const T*>(G.a)[n * G.z_stride + h]) + G.p0[h]);
-  d = expf(-expf(G.p1[h]) * c);
+  log_d = -expf(G.p1[h]) * c;
 }
 
 // (f, i) stands for m -> max(f + m, i); `first` is applied before `then`
@@ -242,7 +242,7 @@ __device__ __forceinline__ float2 max_plus(const float2& first, const float2& th
 // maps gives every token's running maximum.  m_state [slots, H] is read (unless fresh: 0) and written back.
 template <typename T>
 __global__ void __launch_bounds__(256)
-capped_gates_kernel(float* __restrict__ decay, float* __restrict__ coef, float* __restrict__ m_seq, DecayGates G,
+capped_gates_kernel(float* __restrict__ log_decay, float* __restrict__ coef, float* __restrict__ m_seq, DecayGates G,
                     float* __restrict__ m_state, const SeqSpan* __restrict__ seqs, int H) {
   __shared__ float2 part[8];
   __shared__ float last[8];
@@ -274,7 +274,7 @@ capped_gates_kernel(float* __restrict__ decay, float* __restrict__ coef, float* 
     if (lane == 0) before = warp == 0 ? m0 : last[warp - 1];   // exactly the value the token before was given
     if (in) {
       const int64_t at = static_cast<int64_t>(sq.tok0 + t) * H + h;
-      decay[at] = expf(f_log + before - m);
+      log_decay[at] = f_log + before - m;
       coef[at] = expf(i_log - m);
       m_seq[at] = m;
     }
@@ -286,14 +286,14 @@ capped_gates_kernel(float* __restrict__ decay, float* __restrict__ coef, float* 
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-step_sizes_kernel(float* __restrict__ decay, float* __restrict__ coef, DecayGates G, int64_t n_tok, int H) {
+step_sizes_kernel(float* __restrict__ log_decay, float* __restrict__ coef, DecayGates G, int64_t n_tok, int H) {
   const int64_t total = n_tok * H;
   for (int64_t e = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x; e < total;
        e += static_cast<int64_t>(gridDim.x) * blockDim.x) {
     const int64_t n = e / H;
     float d, c;
     step_size<T>(G, n, static_cast<int>(e - n * H), d, c);
-    decay[e] = d;
+    log_decay[e] = d;
     coef[e] = c;
   }
 }
@@ -314,7 +314,7 @@ struct ScanArgs {
   const void* k;
   const void* v;
   int64_t q_stride, k_stride, v_stride;
-  const float* decay;  // [n, H]
+  const float* log_decay;  // [n, H]
   const float* coef;   // [n, H]
   const float* skip;   // [H] or NULL
   float q_scale;
@@ -343,7 +343,7 @@ decay_scan_kernel(const ScanArgs A) {
   const T* q = static_cast<const T*>(A.q) + static_cast<int64_t>(sq.tok0) * A.q_stride + static_cast<int64_t>(g) * dk;
   const T* k = static_cast<const T*>(A.k) + static_cast<int64_t>(sq.tok0) * A.k_stride + static_cast<int64_t>(g) * dk;
   const T* v = static_cast<const T*>(A.v) + static_cast<int64_t>(sq.tok0) * A.v_stride + static_cast<int64_t>(h) * dv + col0;
-  const float* dec = A.decay + static_cast<int64_t>(sq.tok0) * A.H + h;
+  const float* dec = A.log_decay + static_cast<int64_t>(sq.tok0) * A.H + h;
   const float* cof = A.coef + static_cast<int64_t>(sq.tok0) * A.H + h;
   const float skip = A.skip ? A.skip[h] : 0.f;
   float S[RW4];
@@ -371,7 +371,7 @@ decay_scan_kernel(const ScanArgs A) {
       const int tt = e / kScanCols, i = e % kScanCols;
       dst[tt * ROW + 2 * DK + i] = i < ncol ? Cvt<T>::to_f32(v[static_cast<int64_t>(t0 + tt) * A.v_stride + i]) : 0.f;
     }
-    if (tid < n_here) dst[tid * ROW + 2 * DK + kScanCols] = dec[static_cast<int64_t>(t0 + tid) * A.H];
+    if (tid < n_here) dst[tid * ROW + 2 * DK + kScanCols] = expf(dec[static_cast<int64_t>(t0 + tid) * A.H]);
   };
   float* buf0 = sc_sm;
   float* buf1 = sc_sm + kScanChunk * ROW;
@@ -480,6 +480,7 @@ decay_step_kernel(const StepArgs A) {
     if (blockIdx.z == 0 && tid == 0) A.m_seq[n * A.H + h] = m;
   } else {
     step_size<T>(A.gates, n, h, d, c);
+    d = expf(d);
   }
   const T* q = static_cast<const T*>(A.q) + n * A.q_stride + static_cast<int64_t>(g) * dk;
   const T* k = static_cast<const T*>(A.k) + n * A.k_stride + static_cast<int64_t>(g) * dk;
@@ -695,48 +696,48 @@ int b200_silu_glu(void* y, const void* gu, int64_t rows, int ff, int dtype, void
   });
 }
 
-int b200_capped_gates(float* decay, float* coef, float* m_seq, const void* zi, const void* zf, int64_t z_stride,
+int b200_capped_gates(float* log_decay, float* coef, float* m_seq, const void* zi, const void* zf, int64_t z_stride,
                       const float* bias_i, const float* bias_f, float cap, float* m_state, const int32_t* seqs, int n_seqs,
                       int H, int dtype, void* stream) {
   if (n_seqs < 0 || H <= 0 || !(cap > 0.f)) return fail(B200_EINVAL, "b200_capped_gates: bad sizes");
   if (n_seqs == 0) return 0;
-  if (!decay || !coef || !m_seq || !zi || !zf || !bias_i || !bias_f || !m_state || !seqs)
+  if (!log_decay || !coef || !m_seq || !zi || !zf || !bias_i || !bias_f || !m_state || !seqs)
     return fail(B200_EINVAL, "b200_capped_gates: null pointer");
   const DecayGates G{zi, zf, z_stride, bias_i, bias_f, cap, 0};
   return recurrent_by_dtype(dtype, "b200_capped_gates", [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     capped_gates_kernel<T><<<dim3(n_seqs, H), 256, 0, static_cast<cudaStream_t>(stream)>>>(
-        decay, coef, m_seq, G, m_state, reinterpret_cast<const SeqSpan*>(seqs), H);
+        log_decay, coef, m_seq, G, m_state, reinterpret_cast<const SeqSpan*>(seqs), H);
     return check_launch("b200_capped_gates");
   });
 }
 
-int b200_step_sizes(float* decay, float* coef, const void* z, int64_t z_stride, const float* bias, const float* a_log,
+int b200_step_sizes(float* log_decay, float* coef, const void* z, int64_t z_stride, const float* bias, const float* a_log,
                     int64_t n_tok, int H, int dtype, void* stream) {
   if (n_tok < 0 || H <= 0) return fail(B200_EINVAL, "b200_step_sizes: bad sizes");
   if (n_tok == 0) return 0;
-  if (!decay || !coef || !z || !bias || !a_log) return fail(B200_EINVAL, "b200_step_sizes: null pointer");
+  if (!log_decay || !coef || !z || !bias || !a_log) return fail(B200_EINVAL, "b200_step_sizes: null pointer");
   const DecayGates G{z, nullptr, z_stride, bias, a_log, 1.f, 1};
   const unsigned grid = static_cast<unsigned>(std::min<int64_t>((n_tok * H + 255) / 256, kNumSMs * 16));
   return recurrent_by_dtype(dtype, "b200_step_sizes", [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
-    step_sizes_kernel<T><<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(decay, coef, G, n_tok, H);
+    step_sizes_kernel<T><<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(log_decay, coef, G, n_tok, H);
     return check_launch("b200_step_sizes");
   });
 }
 
 int b200_decay_scan(float* o, float* nq, const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v,
-                    int64_t v_stride, const float* decay, const float* coef, const float* skip, float q_scale, float* state,
+                    int64_t v_stride, const float* log_decay, const float* coef, const float* skip, float q_scale, float* state,
                     float* nstate, const int32_t* seqs, int n_seqs, int H, int G, int dk, int dv, int dtype, void* stream) {
   if (n_seqs < 0 || H <= 0 || G <= 0 || H % G || dk <= 0 || dv <= 0) return fail(B200_EINVAL, "b200_decay_scan: bad sizes");
   if (dk > 512) return fail(B200_ESHAPE, "b200_decay_scan: key size %d beyond 512", dk);
   if (n_seqs == 0) return 0;
-  if (!o || !q || !k || !v || !decay || !coef || !state || !seqs || (nstate && !nq))
+  if (!o || !q || !k || !v || !log_decay || !coef || !state || !seqs || (nstate && !nq))
     return fail(B200_EINVAL, "b200_decay_scan: null pointer");
   const int dkt = dk <= 32 ? 32 : (dk <= 64 ? 64 : (dk <= 128 ? 128 : (dk <= 256 ? 256 : 512)));
   const size_t smem = sizeof(float) * 2 * kScanChunk * (2 * static_cast<size_t>(dkt) + kScanCols + 4);
   const dim3 grid(n_seqs, H, (dv + kScanCols - 1) / kScanCols);
-  const ScanArgs A{o, nq, q, k, v, q_stride, k_stride, v_stride, decay, coef, skip, q_scale, state, nstate,
+  const ScanArgs A{o, nq, q, k, v, q_stride, k_stride, v_stride, log_decay, coef, skip, q_scale, state, nstate,
                    reinterpret_cast<const SeqSpan*>(seqs), H, G, dk, dv};
   return recurrent_by_dtype(dtype, "b200_decay_scan", [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;

@@ -1040,7 +1040,7 @@ def _f32_heads(*tensors: torch.Tensor, H: int) -> None:
 @_timed
 def capped_gates(zi: torch.Tensor, zf: torch.Tensor, bias_i: torch.Tensor, bias_f: torch.Tensor, cap: float,
                  m_state: torch.Tensor, seqs: torch.Tensor):
-    """Exponential gates with a soft cap and a running maximum: ``(decay, coef, m)``, fp32 ``[n, H]`` each (see
+    """Exponential gates with a soft cap and a running maximum: ``(log decay, coef, m)``, fp32 ``[n, H]`` each (see
     ``b200_capped_gates``).  ``zi / zf [n, H]`` are column slices of one projection; ``m_state`` fp32 ``[slots, H]`` carries
     the maximum and is updated."""
     _need_cuda(zi, zf, m_state, seqs)
@@ -1051,25 +1051,25 @@ def capped_gates(zi: torch.Tensor, zf: torch.Tensor, bias_i: torch.Tensor, bias_
         raise ValueError("zi and zf are [n, H] slices with one row stride")
     if m_state.dtype != torch.float32 or m_state.shape[1:] != (H,) or not m_state.is_contiguous():
         raise ValueError("m_state is contiguous fp32 [slots, H]")
-    decay, coef, m = torch.empty((3, n, H), dtype=torch.float32, device=zi.device).unbind(0)
-    rc = _lib_().b200_capped_gates(decay.data_ptr(), coef.data_ptr(), m.data_ptr(), zi.data_ptr(), zf.data_ptr(), _rows2(zi),
+    log_decay, coef, m = torch.empty((3, n, H), dtype=torch.float32, device=zi.device).unbind(0)
+    rc = _lib_().b200_capped_gates(log_decay.data_ptr(), coef.data_ptr(), m.data_ptr(), zi.data_ptr(), zf.data_ptr(), _rows2(zi),
                                    bias_i.data_ptr(), bias_f.data_ptr(), float(cap), m_state.data_ptr(), seqs.data_ptr(),
                                    seqs.shape[0], H, DTYPE_ID[zi.dtype], _stream())
     _lib.check_mixers(rc, "b200_capped_gates")
-    return decay, coef, m
+    return log_decay, coef, m
 
 
 @_timed
 def step_sizes(z: torch.Tensor, bias: torch.Tensor, a_log: torch.Tensor):
-    """``dt = softplus(z + bias)``, ``decay = exp(-exp(a_log) dt)``: ``(decay, dt)``, fp32 ``[n, H]``."""
+    """``dt = softplus(z + bias)``: ``(log decay = -exp(a_log) dt, dt)``, fp32 ``[n, H]``."""
     _need_cuda(z)
     n, H = z.shape
     _f32_heads(bias, a_log, H=H)
-    decay, coef = torch.empty((2, n, H), dtype=torch.float32, device=z.device).unbind(0)
-    rc = _lib_().b200_step_sizes(decay.data_ptr(), coef.data_ptr(), z.data_ptr(), _rows2(z), bias.data_ptr(), a_log.data_ptr(),
+    log_decay, coef = torch.empty((2, n, H), dtype=torch.float32, device=z.device).unbind(0)
+    rc = _lib_().b200_step_sizes(log_decay.data_ptr(), coef.data_ptr(), z.data_ptr(), _rows2(z), bias.data_ptr(), a_log.data_ptr(),
                                  n, H, DTYPE_ID[z.dtype], _stream())
     _lib.check_mixers(rc, "b200_step_sizes")
-    return decay, coef
+    return log_decay, coef
 
 
 def _check_decay_inputs(q, k, v, state, nstate, seqs, G: int):
@@ -1088,24 +1088,32 @@ def _check_decay_inputs(q, k, v, state, nstate, seqs, G: int):
     return n, H, dk, dv
 
 
+CHUNK_SCAN_FROM = 16     # tokens of a step's longest portion from which the chunked tensor-core scan serves the step
+
+
 @_timed
-def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, coef: torch.Tensor,
+def decay_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, log_decay: torch.Tensor, coef: torch.Tensor,
                state: torch.Tensor, seqs: torch.Tensor, G: int, q_scale: float = 1.0, skip: Optional[torch.Tensor] = None,
-               nstate: Optional[torch.Tensor] = None):
-    """``S <- decay S + coef k v^T``, ``o = S^T (q_scale q) + skip v`` over each sequence's tokens, and with ``nstate`` the
-    vector recurrence ``n <- decay n + coef k`` and ``n . (q_scale q)``.  ``q / k [n, G*dk]``, ``v [n, H*dv]``, ``decay /
-    coef`` fp32 ``[n, H]``, ``state`` fp32 ``[slots, H, dk, dv]``.  Returns ``(o fp32 [n, H, dv], nq fp32 [n, H] or None)``."""
+               nstate: Optional[torch.Tensor] = None, max_count: int = 0):
+    """``S <- e^log_decay S + coef k v^T``, ``o = S^T (q_scale q) + skip v`` over each sequence's tokens, and with ``nstate``
+    the vector recurrence ``n <- e^log_decay n + coef k`` and ``n . (q_scale q)``.  ``q / k [n, G*dk]``, ``v [n, H*dv]``,
+    ``log_decay / coef`` fp32 ``[n, H]``, ``state`` fp32 ``[slots, H, dk, dv]``.  Returns ``(o fp32 [n, H, dv], nq fp32 [n, H]
+    or None)``.  ``max_count``: the largest token count in ``seqs`` (picks the kernel: bf16 steps with a portion of
+    ``CHUNK_SCAN_FROM`` tokens or more run chunks on the tensor cores, others token by token)."""
     n, H, dk, dv = _check_decay_inputs(q, k, v, state, nstate, seqs, G)
     _f32_heads(skip, H=H)
-    for t in (decay, coef):
+    for t in (log_decay, coef):
         if t.dtype != torch.float32 or tuple(t.shape) != (n, H) or not t.is_contiguous():
-            raise ValueError("decay and coef are contiguous fp32 [n, H]")
+            raise ValueError("log_decay and coef are contiguous fp32 [n, H]")
     o = torch.empty((n, H, dv), dtype=torch.float32, device=q.device)
     nq = torch.empty((n, H), dtype=torch.float32, device=q.device) if nstate is not None else None
-    rc = _lib_().b200_decay_scan(o.data_ptr(), _ptr(nq), q.data_ptr(), _rows2(q), k.data_ptr(), _rows2(k), v.data_ptr(),
-                                 _rows2(v), decay.data_ptr(), coef.data_ptr(), _ptr(skip), float(q_scale), state.data_ptr(),
-                                 _ptr(nstate), seqs.data_ptr(), seqs.shape[0], H, G, dk, dv, DTYPE_ID[q.dtype], _stream())
-    _lib.check_mixers(rc, "b200_decay_scan")
+    lib, dt = _lib_(), DTYPE_ID[q.dtype]
+    chunks = max_count >= CHUNK_SCAN_FROM and lib.b200_decay_chunk_scan_supported(dk, dv, dt)
+    fn = lib.b200_decay_chunk_scan if chunks else lib.b200_decay_scan
+    rc = fn(o.data_ptr(), _ptr(nq), q.data_ptr(), _rows2(q), k.data_ptr(), _rows2(k), v.data_ptr(), _rows2(v),
+            log_decay.data_ptr(), coef.data_ptr(), _ptr(skip), float(q_scale), state.data_ptr(), _ptr(nstate), seqs.data_ptr(),
+            seqs.shape[0], H, G, dk, dv, dt, _stream())
+    _lib.check_mixers(rc, "b200_decay_chunk_scan" if chunks else "b200_decay_scan")
     return o, nq
 
 

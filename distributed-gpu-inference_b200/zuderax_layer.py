@@ -186,8 +186,9 @@ class MatrixMemoryMixer(nn.Module):
                                             q_scale=dk ** -0.5, nstate=n_state, m_state=m_state)
             y = mixer_ops.normalized_head_out(o, nq, m, READOUT_FLOOR, self.norm_w, gate, self.eps, m_state, st.scan_seqs)
         else:
-            decay, coef, m = mixer_ops.capped_gates(zi, zf, self.b_i, self.b_f, self.cap, m_state, st.scan_seqs)
-            o, nq = mixer_ops.decay_scan(q, k, v, decay, coef, S, st.scan_seqs, H, q_scale=dk ** -0.5, nstate=n_state)
+            log_decay, coef, m = mixer_ops.capped_gates(zi, zf, self.b_i, self.b_f, self.cap, m_state, st.scan_seqs)
+            o, nq = mixer_ops.decay_scan(q, k, v, log_decay, coef, S, st.scan_seqs, H, q_scale=dk ** -0.5, nstate=n_state,
+                                         max_count=st.max_count())
             y = mixer_ops.normalized_head_out(o, nq, m, READOUT_FLOOR, self.norm_w, gate, self.eps)
         return F.linear(y, self.w_o)
 
@@ -227,8 +228,9 @@ class StateSpaceMixer(nn.Module):
         if st.max_count() == 1:
             y, _, _ = mixer_ops.decay_step(C, B, x, ("step", dt, self.dt_bias, self.a_log), S, st.scan_seqs, G, skip=self.skip)
         else:
-            decay, coef = mixer_ops.step_sizes(dt, self.dt_bias, self.a_log)
-            y, _ = mixer_ops.decay_scan(C, B, x, decay, coef, S, st.scan_seqs, G, skip=self.skip)
+            log_decay, coef = mixer_ops.step_sizes(dt, self.dt_bias, self.a_log)
+            y, _ = mixer_ops.decay_scan(C, B, x, log_decay, coef, S, st.scan_seqs, G, skip=self.skip,
+                                        max_count=st.max_count())
         return F.linear(mixer_ops.gated_part_norm(y, proj[:, :self.inner], self.norm_w, self.eps, self.parts), self.w_o)
 
 
@@ -384,11 +386,11 @@ def random_checkpoint(config: ZuderaxConfig, seed: int = 0, dtype: torch.dtype =
     def vec(n, s=1.0, mean=0.0):
         return (mean + s * torch.randn(n, generator=g)).to(dtype)
 
-    t: Dict[str, torch.Tensor] = {"embed": torch.randn(config.vocab, W, generator=g).to(dtype)}
+    t: Dict[str, torch.Tensor] = {"embed": (3.0 * torch.randn(config.vocab, W, generator=g)).to(dtype)}
 
     def norm(name):
         t[name], t[name + ".b"] = vec(W, 0.2, 1.2), vec(W, 0.1)
-        t[name + ".alpha"] = (0.5 + 0.3 * torch.rand((), generator=g)).to(dtype)
+        t[name + ".alpha"] = (0.25 + 0.2 * torch.rand((), generator=g)).to(dtype)
 
     for i, layer in enumerate(config.layers):
         if layer.get("weights_of") is not None:

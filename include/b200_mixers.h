@@ -391,28 +391,37 @@ int b200_silu_glu(void* y, const void* gu, int64_t rows, int ff, int dtype, void
 
 /* Capped exponential gates of a step's portions (SeqSpan rows): with sc(z) = cap * tanh(z / cap), i = sc(zi + bias_i),
  * f = log sigmoid(sc(zf + bias_f)) and the running maximum m_t = max(f + m_(t-1), i):
- *   decay = exp(f + m_(t-1) - m_t),  coef = exp(i - m_t),  m_seq = m_t          fp32 [n_tok, H]
+ *   log_decay = f + m_(t-1) - m_t,  coef = exp(i - m_t),  m_seq = m_t            fp32 [n_tok, H]
  * zi, zf: T rows [n_tok, H] with row stride z_stride; biases fp32 [H]; m_state fp32 [slots, H] carries m (0 when the sequence
  * is fresh) and is updated. */
-int b200_capped_gates(float* decay, float* coef, float* m_seq, const void* zi, const void* zf, int64_t z_stride,
+int b200_capped_gates(float* log_decay, float* coef, float* m_seq, const void* zi, const void* zf, int64_t z_stride,
                       const float* bias_i, const float* bias_f, float cap, float* m_state, const int32_t* seqs, int n_seqs,
                       int H, int dtype, void* stream);
 
-/* Step sizes: coef = dt = softplus(z + bias), decay = exp(-exp(a_log) * dt); z T rows [n_tok, H]; bias, a_log fp32 [H]. */
-int b200_step_sizes(float* decay, float* coef, const void* z, int64_t z_stride, const float* bias, const float* a_log,
+/* Step sizes: coef = dt = softplus(z + bias), log_decay = -exp(a_log) * dt; z T rows [n_tok, H]; bias, a_log fp32 [H]. */
+int b200_step_sizes(float* log_decay, float* coef, const void* z, int64_t z_stride, const float* bias, const float* a_log,
                     int64_t n_tok, int H, int dtype, void* stream);
 
 /* Decayed outer-product state per (sequence, head) over the sequence's tokens of this step, in order (SeqSpan rows):
- *   S <- decay[t][h] S + coef[t][h] k_t v_t^T;   o_t = S^T (q_scale q_t) + skip[h] v_t              (skip may be NULL)
- *   n <- decay[t][h] n + coef[t][h] k_t;         nq_t = n . (q_scale q_t)                           (nstate NULL: no n)
- * q, k: T rows of G*dk (head h reads head h / (H / G)), v: T rows of H*dv, each with its row stride; decay, coef fp32
- * [n_tok, H]; skip fp32 [H]; state fp32 [slots, H, dk, dv] and nstate fp32 [slots, H, dk], read unless the sequence is fresh
+ *   S <- e^log_decay[t][h] S + coef[t][h] k_t v_t^T;   o_t = S^T (q_scale q_t) + skip[h] v_t        (skip may be NULL)
+ *   n <- e^log_decay[t][h] n + coef[t][h] k_t;         nq_t = n . (q_scale q_t)                     (nstate NULL: no n)
+ * q, k: T rows of G*dk (head h reads head h / (H / G)), v: T rows of H*dv, each with its row stride; log_decay, coef
+ * fp32 [n_tok, H]; skip fp32 [H]; state fp32 [slots, H, dk, dv] and nstate fp32 [slots, H, dk], read unless the sequence is fresh
  * and written back; o fp32 [n_tok, H, dv], nq fp32 [n_tok, H].  dk <= 512. */
 int b200_decay_scan(float* o, float* nq, const void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v,
-                    int64_t v_stride, const float* decay, const float* coef, const float* skip, float q_scale, float* state,
+                    int64_t v_stride, const float* log_decay, const float* coef, const float* skip, float q_scale, float* state,
                     float* nstate, const int32_t* seqs, int n_seqs, int H, int G, int dk, int dv, int dtype, void* stream);
 
-/* The same for steps whose sequences bring ONE token each (row n = sequence n), decay and coef formed on the way:
+/* The same in chunks of 64 tokens on the tensor cores (bf16, dk <= 256): q, k and v enter the products as they are, fp32
+ * operands (state, pair weights, weighted keys) as the sum of two bf16 numbers, accumulation and state are fp32.  For steps
+ * that carry prompt portions; any portion length is served. */
+int b200_decay_chunk_scan_supported(int dk, int dv, int dtype);
+int b200_decay_chunk_scan(float* o, float* nq, const void* q, int64_t q_stride, const void* k, int64_t k_stride,
+                          const void* v, int64_t v_stride, const float* log_decay, const float* coef, const float* skip,
+                          float q_scale, float* state, float* nstate, const int32_t* seqs, int n_seqs, int H, int G, int dk,
+                          int dv, int dtype, void* stream);
+
+/* The same for steps whose sequences bring ONE token each (row n = sequence n), log_decay and coef formed on the way:
  * gate_kind 0: b200_capped_gates with za = zi, zb = zf, p0 = bias_i, p1 = bias_f; m_seq [n_tok, H] receives the new running
  * maximum, m_state is only read (b200_normalized_head_out stores it); gate_kind 1: b200_step_sizes with za = z, p0 = bias,
  * p1 = a_log (zb, m_seq, m_state NULL). */

@@ -1,0 +1,655 @@
+"""GPU: the Zuderax model class on the ragged step engine against the plain float64 statement in oracle/zuderax_ref.py.
+
+Small configurations with random weights; sizes are chosen so that nothing is a multiple of a warp, a page, a key tile or a
+scan chunk by accident (one head, key sizes 2 / 6 / 33 / 40, value sizes 3 / 10 / 33 / 72, state groups 1 / 2 / 3, norm parts
+that cut heads in two, 1 / 2 / 4 / 5 taps, windows of 1, 9, 19 and longer than the sequence, group counts 1 / 2 / 3 / 4 with 1
+to all kept, layers without a feed-forward, layers that run another layer's weights).  Where random weights would hide a fault
+the inputs are made so that it shows: one key dominates just inside and just outside a window, gates saturate, decays are
+close to 1 and close to 0, one far key among hundreds is the only one a query matches.
+"""
+import math
+
+import pytest
+import torch
+
+import dgi_b200  # noqa: F401
+from oracle import zuderax_ref as R
+
+pytestmark = pytest.mark.gpu
+
+DEV = "cuda:0"
+F64 = torch.float64
+
+
+def latent(heads, dim, rot_dim, vdim, rank, size, base=10000.0, scale=None):
+    return {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": rank, "mask": {"size": size},
+            "scale": scale or 1.0 / math.sqrt(dim + rot_dim), "rot": {"base": base, "dims": rot_dim}}
+
+
+def mlstm(heads, dim, vdim, cap):
+    return {"heads": heads, "dim": dim, "vdim": vdim, "gate_cap": cap}
+
+
+def mamba2(heads, vdim, state, groups, conv, parts):
+    return {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "conv": conv, "norm_groups": parts}
+
+
+def dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def moe(experts, top, ff, groups=1, keep=1, scale=1.0, shared=None):
+    spec = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top, "scale": scale,
+                                                            "groups": {"count": groups, "keep": keep}}}
+    if shared:
+        spec["shared"] = {"ff": shared}
+    return spec
+
+
+def layer(kind, mixer, mlp, of=None):
+    out = {"type": kind, "mixer": mixer, "mlp": mlp}
+    if of is not None:
+        out["weights_of"] = of
+    return out
+
+
+_A0 = layer("latent_attention", latent(3, 12, 6, 20, 22, 9, base=50.0, scale=0.3), moe(6, 3, 20, 3, 2, 1.7, shared=12))
+_A1 = layer("mlstm", mlstm(2, 6, 10, 5.0), dense(24))
+_A2 = layer("mamba2", mamba2(6, 10, 7, 3, 5, 4), None)
+CFG_A = {   # sizes off every grid
+    "architecture": "Zuderax", "width": 56, "vocab": 53, "norm": {"eps": 1e-5}, "logit_scale": 0.3,
+    "layers": [_A0, _A1, _A2, dict(_A1, weights_of=1), dict(_A0, weights_of=0), dict(_A2, weights_of=2),
+               layer("mlstm", mlstm(3, 33, 3, 8.0), moe(5, 5, 8, shared=20)),
+               layer("mamba2", mamba2(1, 33, 40, 1, 1, 1), moe(4, 1, 16, 4, 1, 0.5))],
+}
+CFG_B = {   # sizes the tensor-core kernels and the grouped expert GEMM take in 16-bit storage
+    "architecture": "Zuderax", "width": 64, "vocab": 41, "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+    "layers": [
+        layer("mlstm", mlstm(4, 32, 48, 10.0), moe(8, 2, 32, 2, 1, 2.5, shared=24)),
+        layer("latent_attention", latent(10, 16, 16, 24, 48, 19, base=200.0), dense(96)),
+        layer("mamba2", mamba2(4, 32, 64, 2, 4, 2), dense(40)),
+        layer("latent_attention", latent(2, 32, 8, 16, 72, 40), None),
+        layer("mamba2", mamba2(8, 16, 16, 1, 2, 8), moe(8, 4, 16, 4, 4, 1.0, shared=16)),
+        layer("mlstm", mlstm(1, 80, 72, 3.0), None),
+        layer("mamba2", mamba2(2, 64, 128, 2, 3, 1), moe(4, 2, 48, 2, 2)),
+    ],
+}
+CFG_C = {   # the smallest of everything
+    "architecture": "Zuderax", "width": 8, "vocab": 11, "norm": {"eps": 1e-6},
+    "layers": [layer("latent_attention", latent(1, 2, 2, 2, 4, 1), moe(1, 1, 8)),
+               layer("mlstm", mlstm(1, 2, 1, 1.0), None),
+               layer("mamba2", mamba2(1, 1, 1, 1, 1, 1), moe(2, 2, 8, 2, 2))],
+}
+CFG_D = {   # recurrences only: no pages at all
+    "architecture": "Zuderax", "width": 48, "vocab": 37, "norm": {"eps": 1e-6},
+    "layers": [layer("mamba2", mamba2(3, 16, 32, 1, 4, 3), dense(64)), layer("mlstm", mlstm(2, 16, 16, 15.0), dense(64))],
+}
+
+
+def build(cfg_raw, dtype=torch.float32, seed=0, max_tokens=512, max_seqs=4, tensors=None):
+    from dgi_b200 import zuderax_layer as Z
+    from dgi_b200.ragged_engine import RaggedStepEngine
+
+    cfg = Z.ZuderaxConfig.from_dict(cfg_raw)
+    tensors = tensors or Z.random_checkpoint(cfg, seed=seed)
+    shards = Z.build_shards(cfg, tensors, [(0, cfg.num_hidden_layers)], DEV, dtype)
+    return RaggedStepEngine(shards, max_tokens=max_tokens, max_seqs=max_seqs), tensors
+
+
+def tokens(n, vocab, seed):
+    return torch.randint(0, vocab, (n,), generator=torch.Generator().manual_seed(seed)).tolist()
+
+
+def whole(engine, rid, toks, want=None):
+    want = list(range(len(toks))) if want is None else want
+    out = engine.step([(rid, toks, want)]).cpu()
+    engine.finish(rid)
+    return out
+
+
+def close(got, ref, tol):
+    err = (got.to(F64) - ref.to(F64)).abs().max().item()
+    assert err <= tol * max(1.0, ref.abs().max().item()), f"max abs error {err}"
+
+
+def rounding_close(got, ref, median=0.05, tail=0.15, tail_share=0.2):
+    """16-bit storage against a wider statement, row by row (error rms over the statement's rms): the typical row is within
+    rounding; a few rows may differ more, where rounding flips an expert's choice, but not many."""
+    row = (got.to(F64) - ref.to(F64)).pow(2).mean(dim=1).sqrt() / ref.to(F64).pow(2).mean().sqrt()
+    assert row.median() <= median, f"median row error {row.median().item()}"
+    assert (row > tail).to(F64).mean() <= tail_share, f"rows over {tail}: {(row > tail).sum().item()} of {row.numel()}"
+
+
+def seqs_of(spans):
+    return torch.tensor(spans, dtype=torch.int32, device=DEV)
+
+
+DT = pytest.mark.parametrize("dt,tol", [(torch.float32, 3e-6), (torch.bfloat16, 1e-2)], ids=["fp32", "bf16"])
+
+
+# ---- elementwise pieces ----------------------------------------------------------------------------------------------
+@DT
+@pytest.mark.parametrize("n,W", [(5, 56), (3, 7), (70, 128)])
+def test_residual_update_with_the_next_dynamic_tanh_norm(dt, tol, n, W):
+    from dgi_b200 import mixer_ops as M
+
+    g = torch.Generator().manual_seed(W)
+    x = 4.0 * torch.randn(n, W, generator=g)
+    y = torch.randn(n, W + 3, generator=g).to(dt)[:, :W]
+    w, b = torch.randn(W, generator=g).to(dt), torch.randn(W, generator=g).to(dt)
+    for branch in (y, y.float(), None):
+        xd = x.to(DEV).clone()
+        out = M.residual_dyn_tanh(xd, branch.to(DEV) if branch is not None else None, (w.to(DEV), b.to(DEV), 0.37))
+        want = x.to(F64) + (branch.to(F64) if branch is not None else 0)
+        close(xd.cpu(), want, 1e-6)                                    # the residual stays fp32
+        close(out.cpu(), R.dyn_tanh(want, torch.tensor(0.37, dtype=F64), w.to(F64), b.to(F64)), tol)
+        assert out.dtype == dt
+    xd = x.to(DEV).clone()
+    assert M.residual_dyn_tanh(xd, y.to(DEV)) is None
+    close(xd.cpu(), x.to(F64) + y.to(F64), 1e-6)
+
+
+@DT
+@pytest.mark.parametrize("ff", [5, 16, 40])
+def test_silu_glu(dt, tol, ff):
+    from dgi_b200 import mixer_ops as M
+
+    gu = 3.0 * torch.randn(9, 2 * ff, generator=torch.Generator().manual_seed(ff)).to(dt)
+    close(M.silu_glu(gu.to(DEV)).cpu(), R.silu(gu[:, :ff].to(F64)) * gu[:, ff:].to(F64), tol)
+
+
+@DT
+@pytest.mark.parametrize("C,taps,bias", [(10, 4, True), (33, 1, True), (64, 4, True), (128, 3, False), (40, 8, True), (12, 11, True)])
+def test_causal_convolution_with_bias_over_portions(dt, tol, C, taps, bias):
+    from dgi_b200 import mixer_ops as M
+
+    g = torch.Generator().manual_seed(C + taps)
+    x = torch.randn(150, C + 6, generator=g).to(dt)[:, 2:2 + C] if C % 4 else torch.randn(150, C, generator=g).to(dt)
+    w = (torch.randn(C, taps, generator=g) / math.sqrt(taps)).to(dt)
+    b = torch.randn(C, generator=g).to(dt) if bias else None
+    want = R.silu(R.causal_conv(x.to(F64), w.to(F64), b.to(F64) if bias else torch.zeros(C, dtype=F64)))
+    tail = torch.full((3, taps - 1, C), float("nan"), device=DEV)       # a fresh sequence never reads its slot
+    dev, at, got = x.to(DEV), 0, []
+    for cut in (70, 1, 2, 1, 66, 3, 7):                                  # portions shorter than the taps, longer than a run
+        got.append(M.causal_conv_silu(dev[at:at + cut], w.to(DEV), tail, seqs_of([(0, cut, 1, int(at == 0))]), cut,
+                                      bias=b.to(DEV) if bias else None))
+        at += cut
+    close(torch.cat(got).cpu(), want, tol)
+
+
+@DT
+@pytest.mark.parametrize("H,dr,rank,dims", [(3, 6, 22, 6), (10, 16, 48, 16), (1, 4, 5, 2), (2, 2, 40, 0)])
+def test_latent_rows_with_half_split_rotary_pairs(dt, tol, H, dr, rank, dims):
+    from dgi_b200 import mixer_ops as M, vatazen_layer as Vz
+
+    g = torch.Generator().manual_seed(H + rank)
+    n, bs, nb = 21, 16, 3
+    q, dkv = torch.randn(n, H, dr, generator=g).to(dt), torch.randn(n, rank + dr, generator=g).to(dt)
+    w = (1.0 + 0.2 * torch.randn(rank, generator=g)).to(dt)
+    pos = torch.randint(0, 5000, (n,), generator=g).to(torch.int32)
+    slots = torch.randperm(nb * bs, generator=g)[:n].to(torch.int64)
+    freqs, _ = Vz.yarn_frequencies(dims, 300.0, None)
+    pool = torch.zeros((nb, 1, bs, rank + dr), dtype=dt, device=DEV)
+    out = torch.empty((n, H, dr), dtype=dt, device=DEV)
+    M.latent_rotary_append(q.to(DEV), out, dkv.to(DEV), w.to(DEV), 1e-5, freqs.to(DEV) if dims else None, 1.0, pool, slots.to(DEV),
+                           pos.to(DEV), interleaved=False)
+    close(out.cpu(), R.rotate_half(q.to(F64), pos, dims, 300.0), tol)
+    rows = pool.view(-1, rank + dr)[slots.to(DEV)].cpu()
+    close(rows[:, :rank], R.rms(dkv[:, :rank].to(F64), 1e-5) * w.to(F64), tol)
+    close(rows[:, rank:], R.rotate_half(dkv[:, rank:].to(F64), pos, dims, 300.0), tol)
+
+
+# ---- recurrences -------------------------------------------------------------------------------------------------------
+def test_capped_gates_running_maximum_over_portions_and_slots():
+    from dgi_b200 import mixer_ops as M
+
+    g = torch.Generator().manual_seed(3)
+    n, H, cap = 700, 3, 6.0
+    z = 4.0 * torch.randn(n, 2 * H + 1, generator=g)
+    z[:, 0] -= torch.linspace(0, 12, n)          # head 0: input gates die away, the maximum decays with f (and starts at 0)
+    z[400, 1] = 60.0                             # head 1: one saturated gate in the middle
+    b_i, b_f = torch.randn(H, generator=g), 2.0 + torch.randn(H, generator=g)
+    i, f = R.capped_gates((z[:, :H] + b_i).to(F64), (z[:, H:2 * H] + b_f).to(F64), cap)
+    m, want_m, want_d, want_c = torch.zeros(H, dtype=F64), [], [], []
+    for t in range(n):
+        new = torch.maximum(f[t] + m, i[t])
+        want_d.append(f[t] + m - new)
+        want_c.append(torch.exp(i[t] - new))
+        want_m.append(new)
+        m = new
+    want_m, want_d, want_c = torch.stack(want_m), torch.stack(want_d), torch.stack(want_c)
+    state = torch.full((4, H), 55.0, device=DEV)
+    dev, at = z.to(DEV), 0
+    for cut in (300, 1, 2, 33, 256, 108):        # beside a one-token sequence of its own in another slot
+        zz = torch.cat([dev[at:at + cut], dev[:1]])
+        d, c, mm = M.capped_gates(zz[:, :H], zz[:, H:2 * H], b_i.to(DEV), b_f.to(DEV), cap, state,
+                                  seqs_of([(0, cut, 2, int(at == 0)), (cut, 1, 0, 1)]))
+        for got, want in ((d, want_d), (c, want_c), (mm, want_m)):
+            close(got[:cut].cpu(), want[at:at + cut], 5e-6)
+            close(got[cut:].cpu(), want[:1], 5e-6)
+        at += cut
+    close(state[2].cpu(), want_m[-1], 5e-6)
+    assert (state[1] == 55.0).all() and (state[3] == 55.0).all()
+
+
+def _scan_case(H, G, dk, dv, n, dt, seed, near_one=False):
+    g = torch.Generator().manual_seed(seed)
+    q, k = torch.randn(n, G * dk, generator=g).to(dt), (torch.randn(n, G * dk, generator=g) / math.sqrt(dk)).to(dt)
+    v = torch.randn(n, H * dv, generator=g).to(dt)
+    decay = torch.rand(n, H, generator=g) * 0.01 + 0.99 if near_one else torch.rand(n, H, generator=g)
+    decay[n // 3] = 0.0                                       # everything before this token is forgotten
+    coef = torch.rand(n, H, generator=g) * 2.0
+    skip = torch.randn(H, generator=g)
+    return q, k, v, decay, coef, skip
+
+
+def _scan_reference(q, k, v, decay, coef, skip, H, G, dk, dv, scale):
+    n = q.shape[0]
+    of = torch.arange(H) // (H // G)
+    Q, K, V = q.to(F64).reshape(n, G, dk)[:, of] * scale, k.to(F64).reshape(n, G, dk)[:, of], v.to(F64).reshape(n, H, dv)
+    S, N, o, nq = torch.zeros(H, dk, dv, dtype=F64), torch.zeros(H, dk, dtype=F64), [], []
+    for t in range(n):
+        d, c = decay[t].to(F64), coef[t].to(F64)
+        S = d[:, None, None] * S + (c[:, None] * K[t])[:, :, None] * V[t][:, None, :]
+        N = d[:, None] * N + c[:, None] * K[t]
+        o.append(torch.einsum("hkv,hk->hv", S, Q[t]) + skip.to(F64)[:, None] * V[t])
+        nq.append((N * Q[t]).sum(-1))
+    return torch.stack(o), torch.stack(nq), S, N
+
+
+SCANS = [(3, 3, 6, 10), (4, 2, 33, 3), (6, 1, 40, 72), (2, 2, 128, 64), (1, 1, 200, 40), (4, 4, 64, 128), (2, 1, 16, 16),
+         (2, 2, 300, 33), (8, 2, 128, 64), (2, 2, 256, 128)]
+
+
+@pytest.mark.parametrize("H,G,dk,dv", SCANS)
+@pytest.mark.parametrize("dt,near_one", [(torch.float32, False), (torch.bfloat16, False), (torch.bfloat16, True), (torch.float16, True)],
+                         ids=["fp32", "bf16", "bf16-slow-decay", "fp16-slow-decay"])
+@pytest.mark.parametrize("chunks", [False, True], ids=["tokens", "chunks"])
+def test_decayed_outer_product_state_over_portions_beside_another_sequence(H, G, dk, dv, dt, near_one, chunks):
+    from dgi_b200 import mixer_ops as M
+
+    if chunks and (dt != torch.bfloat16 or dk > 256):
+        pytest.skip("the chunked scan serves bf16 and key sizes up to 256")
+    n = 330
+    q, k, v, decay, coef, skip = _scan_case(H, G, dk, dv, n, dt, H * dk + dv, near_one)
+    want, want_nq, want_S, want_N = _scan_reference(q, k, v, decay, coef, skip, H, G, dk, dv, 0.7)
+    state = torch.full((3, H, dk, dv), float("nan"), device=DEV)      # a fresh sequence never reads its slot
+    nstate = torch.full((3, H, dk), float("nan"), device=DEV)
+    dq, dk_, dv_, dd, dc = (t.to(DEV) for t in (q, k, v, torch.log(decay), coef))      # one log decay is -inf
+    at, got, got_nq = 0, [], []
+    # what 16-bit inputs allow: they are exact here, and everything between them and the read-outs is 32-bit (or its
+    # equivalent in split 16-bit products)
+    tol = 2e-5 if dt == torch.float32 else 6e-5
+    for cut in (150, 1, 2, 63, 64, 7, 43):
+        cat = lambda t: torch.cat([t[:5], t[at:at + cut]])            # noqa: E731  a second, fresh sequence in front
+        o, nq = M.decay_scan(cat(dq), cat(dk_), cat(dv_), cat(dd).contiguous(), cat(dc).contiguous(), state,
+                             seqs_of([(0, 5, 0, 1), (5, cut, 2, int(at == 0))]), G, q_scale=0.7, skip=skip.to(DEV), nstate=nstate, max_count=64 if chunks else 0)
+        close(o[:5].cpu(), want[:5], tol)
+        close(nq[:5].cpu(), want_nq[:5], tol)
+        got.append(o[5:])
+        got_nq.append(nq[5:])
+        at += cut
+    close(torch.cat(got).cpu(), want, tol)
+    close(torch.cat(got_nq).cpu(), want_nq, tol)
+    close(state[2].cpu(), want_S, tol)
+    close(nstate[2].cpu(), want_N, tol)
+    assert torch.isnan(state[1]).all() and torch.isnan(nstate[1]).all()
+
+
+@pytest.mark.parametrize("H,G,dk,dv", SCANS)
+@pytest.mark.parametrize("dt", [torch.float32, torch.bfloat16], ids=["fp32", "bf16"])
+def test_single_token_steps_equal_the_scan(H, G, dk, dv, dt):
+    """Both gate sources; sequences in shuffled slots, one of them fresh."""
+    from dgi_b200 import mixer_ops as M
+
+    g = torch.Generator().manual_seed(dk + dv)
+    n = 5
+    q, k, v, _, _, skip = _scan_case(H, G, dk, dv, n, dt, 7)
+    z = (2.0 * torch.randn(n, 2 * H, generator=g)).to(dt)
+    p0, p1 = torch.randn(H, generator=g), torch.randn(H, generator=g)
+    spans = seqs_of([(0, 1, 3, 0), (1, 1, 0, 1), (2, 1, 5, 0), (3, 1, 1, 0), (4, 1, 2, 0)])
+    state0 = torch.randn(6, H, dk, dv, generator=g).to(DEV)
+    n0, m0 = torch.randn(6, H, dk, generator=g).to(DEV), torch.randn(6, H, generator=g).to(DEV)
+    dev = [t.to(DEV) for t in (q, k, v, z, p0, p1, skip)]
+    dq, dkk, dvv, dz, dp0, dp1, dskip = dev
+    a, b = [t.clone() for t in (state0, n0, m0)], [t.clone() for t in (state0, n0, m0)]
+    logd, coef, m = M.capped_gates(dz[:, :H], dz[:, H:], dp0, dp1, 4.0, a[2], spans)
+    o, nq = M.decay_scan(dq, dkk, dvv, logd, coef, a[0], spans, G, q_scale=0.6, nstate=a[1])
+    o2, nq2, m2 = M.decay_step(dq, dkk, dvv, ("capped", dz[:, :H], dz[:, H:], dp0, dp1, 4.0), b[0], spans, G, q_scale=0.6,
+                               nstate=b[1], m_state=b[2])
+    for x, y in ((o, o2), (nq, nq2), (m, m2), (a[0], b[0]), (a[1], b[1])):
+        close(y.cpu(), x.cpu(), 2e-5)
+    assert torch.equal(b[2], m0)                         # only read; the read-out norm stores it
+    w, gate = torch.ones(H * dv, dtype=dt, device=DEV), torch.zeros(n, H * dv, dtype=dt, device=DEV)
+    M.normalized_head_out(o2, nq2, m2, 1e-6, w, gate, 1e-6, b[2], spans)
+    close(b[2].cpu(), a[2].cpu(), 1e-6)
+    a, b = state0.clone(), state0.clone()
+    logd, coef = M.step_sizes(dz[:, :H], dp0, dp1)
+    close(coef.cpu(), R.softplus(z[:, :H].to(F64) + p0.to(F64)), 3e-6)
+    close(logd.cpu(), -torch.exp(p1.to(F64)) * R.softplus(z[:, :H].to(F64) + p0.to(F64)), 3e-6)
+    o, _ = M.decay_scan(dq, dkk, dvv, logd, coef, a, spans, G, skip=dskip)
+    o2, _, _ = M.decay_step(dq, dkk, dvv, ("step", dz[:, :H], dp0, dp1), b, spans, G, skip=dskip)
+    close(o2.cpu(), o.cpu(), 2e-5)
+    close(b.cpu(), a.cpu(), 2e-5)
+
+
+def test_matrix_memory_from_gates_to_read_out_against_the_statement():
+    """The whole chain in fp32, with read-outs on both sides of the denominator's maximum."""
+    from dgi_b200 import mixer_ops as M
+
+    g = torch.Generator().manual_seed(9)
+    n, H, dk, dv, cap, eps = 90, 3, 12, 20, 7.0, 1e-5
+    q, k, v = torch.randn(n, H * dk, generator=g), torch.randn(n, H * dk, generator=g), torch.randn(n, H * dv, generator=g)
+    k[:, :dk] *= 0.01                                      # head 0: |n.q| stays below exp(-m)
+    zi, zf = torch.randn(n, H, generator=g) - 2.0, torch.randn(n, H, generator=g) + 2.0
+    zeros = torch.zeros(H)
+    i, f = R.capped_gates(zi.to(F64), zf.to(F64), cap)
+    want, (S, N, m_end) = R.matrix_memory(q.to(F64).reshape(n, H, dk) * dk ** -0.5, k.to(F64).reshape(n, H, dk), v.to(F64).reshape(n, H, dv), i, f)
+    w, gate = torch.randn(H * dv, generator=g), torch.randn(n, H * dv, generator=g)
+    want = R.rms(want, eps).reshape(n, H * dv) * w.to(F64) * torch.sigmoid(gate.to(F64))
+    state, ns, ms = torch.empty(1, H, dk, dv, device=DEV), torch.empty(1, H, dk, device=DEV), torch.empty(1, H, device=DEV)
+    z = torch.cat([zi, zf], dim=1).to(DEV)
+    spans = seqs_of([(0, n, 0, 1)])
+    logd, coef, m = M.capped_gates(z[:, :H], z[:, H:], zeros.to(DEV), zeros.to(DEV), cap, ms, spans)
+    o, nq = M.decay_scan(q.to(DEV), k.to(DEV), v.to(DEV), logd, coef, state, spans, H, q_scale=dk ** -0.5, nstate=ns)
+    assert (nq[:, 0].abs() < torch.exp(-m[:, 0])).all() and (nq[:, 1:].abs() > torch.exp(-m[:, 1:])).any()
+    close(M.normalized_head_out(o, nq, m, 1e-6, w.to(DEV), gate.to(DEV), eps).cpu(), want, 2e-5)
+    close(state[0].cpu(), S, 1e-5)
+    close(ms[0].cpu(), m_end, 1e-5)
+
+
+@DT
+@pytest.mark.parametrize("inner,parts", [(60, 4), (33, 1), (512, 2), (1200, 1), (8, 8)])
+def test_gated_norm_in_parts(dt, tol, inner, parts):
+    from dgi_b200 import mixer_ops as M
+
+    g = torch.Generator().manual_seed(inner)
+    y, z = torch.randn(7, inner, generator=g), torch.randn(7, inner + 5, generator=g).to(dt)[:, :inner]
+    y[:, :inner // parts] *= 30.0                           # one part must not scale the others
+    w = torch.randn(inner, generator=g).to(dt)
+    want = R.rms((y.to(F64) * R.silu(z.to(F64))).reshape(7, parts, -1), 1e-5).reshape(7, inner) * w.to(F64)
+    close(M.gated_part_norm(y.to(DEV), z.to(DEV), w.to(DEV), 1e-5, parts).cpu(), want, tol)
+
+
+# ---- routing -------------------------------------------------------------------------------------------------------------
+@pytest.mark.parametrize("E,top,groups,keep,extra", [(6, 3, 3, 2, 1), (8, 2, 4, 1, 0), (12, 12, 1, 1, 1), (5, 1, 5, 3, 1), (64, 6, 8, 3, 2), (1, 1, 1, 1, 1)])
+def test_sigmoid_routing_with_group_sums_and_negative_choice_scores(E, top, groups, keep, extra):
+    from dgi_b200 import mixer_ops as M
+
+    g = torch.Generator().manual_seed(E)
+    z = 2.0 * torch.randn(203, E + extra, generator=g)
+    corr = torch.randn(E, generator=g) - 1.5                # choice scores on both sides of zero
+    ids, w = M.sigmoid_group_topk(z.to(DEV), corr.to(DEV), E, top, groups, keep, 1.7)
+    want_ids, want_w = R.route(z[:, :E].to(F64), corr.to(F64), top, groups, keep, 1.7)
+    assert torch.equal(ids.cpu().to(torch.int64), want_ids)
+    close(w.cpu(), want_w, 1e-6)
+    ids, w = M.sigmoid_group_topk(z.to(DEV), None, E, top, groups, keep, 1.0)
+    want_ids, want_w = R.route(z[:, :E].to(F64), None, top, groups, keep, 1.0)
+    assert torch.equal(ids.cpu().to(torch.int64), want_ids)
+
+
+def test_a_group_wins_by_the_sum_of_its_two_best_not_by_its_best():
+    from dgi_b200 import mixer_ops as M
+
+    s = torch.tensor([[0.9, 0.1, 0.1, 0.6, 0.6, 0.1]])       # groups of three: 0.9 + 0.1 against 0.6 + 0.6
+    ids, w = M.sigmoid_group_topk(torch.logit(s).to(DEV), None, 6, 2, 2, 1, 1.0)
+    assert sorted(ids[0].tolist()) == [3, 4]
+    close(w.cpu(), torch.full((1, 2), 0.6), 1e-6)            # scores, not renormalised
+
+
+@pytest.mark.parametrize("n,E,W", [(45, 5, 56), (3000, 9, 96), (2500, 12, 33)])
+@pytest.mark.parametrize("dt", [torch.float32, torch.bfloat16], ids=["fp32", "bf16"])
+def test_router_logits_of_16_bit_rows_do_not_depend_on_the_batch(n, E, W, dt):
+    from dgi_b200 import mixer_ops as M
+
+    g = torch.Generator().manual_seed(n)
+    x, w, b = torch.randn(n, W, generator=g).to(dt), torch.randn(E, W, generator=g), torch.randn(E, generator=g)
+    got = M.router_logits(x.to(DEV), w.to(DEV), b.to(DEV))
+    close(got.cpu(), x.to(F64) @ w.to(F64).T + b.to(F64), 2e-6 * W ** 0.5)
+    for row in (0, n // 2, n - 1):
+        one = M.router_logits(x[row:row + 1].contiguous().to(DEV), w.to(DEV), b.to(DEV))
+        assert torch.equal(one[0], got[row])
+
+
+@pytest.mark.parametrize("spec,W", [(moe(6, 3, 20, 3, 2, 1.7, shared=12), 56), (moe(8, 2, 32, 2, 1, 2.5, shared=24), 64),
+                                    (moe(1, 1, 8), 16), (moe(4, 4, 48, 2, 2, 0.5), 64), (moe(5, 2, 7, shared=9), 33)])
+@pytest.mark.parametrize("dt", [torch.float32, torch.bfloat16], ids=["fp32", "bf16"])
+def test_routed_feed_forward_with_gated_shared_expert_and_fused_residual(dt, spec, W):
+    from dgi_b200 import zuderax_layer as Z
+
+    cfg = {"architecture": "Zuderax", "width": W, "vocab": 5, "norm": {"eps": 1e-6},
+           "layers": [layer("mlstm", mlstm(1, 4, 4, 2.0), spec)]}
+    t = {k[7:]: v for k, v in Z.random_checkpoint(Z.ZuderaxConfig.from_dict(cfg), seed=W).items() if k.startswith("l0.mlp.")}
+    g = torch.Generator().manual_seed(1)
+    h, x = torch.randn(83, W, generator=g).to(dt), torch.randn(83, W, generator=g)
+    w, b = torch.randn(W, generator=g).to(dt), torch.randn(W, generator=g).to(dt)
+    want = x.to(F64) + R.moe(h.to(F64), spec, {k: v.to(F64) for k, v in t.items()})
+    xd = x.to(DEV).clone()
+    out = Z.SigmoidGroupMoE(spec, t, DEV, dt)(h.to(DEV), xd, (w.to(DEV), b.to(DEV), 0.4))
+    if dt == torch.float32:
+        close(xd.cpu(), want, 1e-5)
+        close(out.cpu(), R.dyn_tanh(want, torch.tensor(0.4, dtype=F64), w.to(F64), b.to(F64)), 1e-5)
+    else:
+        rounding_close(xd.cpu(), want, median=0.02, tail=0.05, tail_share=0.05)
+
+
+# ---- attention edges -------------------------------------------------------------------------------------------------------
+def _edge_model(window, rank=24, heads=2):
+    """A one-layer model whose scores are one number per token: the query is a constant and the latent carries the token's
+    own mark, so a single marked token takes all the weight wherever it is visible."""
+    W, dn, dr, dv = 32, 8, 4, 8
+    cfg = {"architecture": "Zuderax", "width": W, "vocab": 4, "norm": {"eps": 1e-6},
+           "layers": [layer("latent_attention", latent(heads, dn, dr, dv, rank, window, scale=1.0), None)]}
+    g = torch.Generator().manual_seed(window)
+    f = lambda *s: torch.randn(*s, generator=g) / math.sqrt(s[-1])    # noqa: E731
+    t = {"embed": torch.zeros(4, W), "head": f(4, W)}
+    t["embed"][:, 0] = 3.0                                            # every token: a constant channel
+    t["embed"][1, 1], t["embed"][0, 2], t["embed"][2, 3], t["embed"][3, 4] = 3.0, 3.0, 3.0, 3.0
+    for name in ("l0.norm1", "final.norm"):
+        t[name], t[name + ".b"], t[name + ".alpha"] = torch.ones(W), torch.zeros(W), torch.tensor(1.0)
+    q, uk, dkv = torch.zeros(heads * (dn + dr), W), torch.zeros(heads * dn, rank), torch.zeros(rank + dr, W)
+    for h in range(heads):
+        q[h * (dn + dr), 0] = 4.0                                     # query: constant
+        uk[h * dn, 1] = 4.0                                           # key: latent channel 1, which token 1 carries
+    for j in range(5):
+        dkv[j, j] = 1.0
+    t.update({"l0.mix.q": q, "l0.mix.uk": uk, "l0.mix.dkv": dkv, "l0.mix.dkv.norm": torch.ones(rank),
+              "l0.mix.uv": f(heads * dv, rank), "l0.mix.o": f(W, heads * dv)})
+    return cfg, {k: v.to(torch.bfloat16) for k, v in t.items()}
+
+
+@pytest.mark.parametrize("dt,tol", [(torch.float32, 2e-5), (torch.bfloat16, 0.03)], ids=["fp32", "bf16"])
+@pytest.mark.parametrize("window", [1, 2, 15, 16, 17, 33, 64, 100])
+def test_a_dominating_key_just_inside_and_just_outside_the_window_in_prompts_and_decoding(dt, tol, window):
+    cfg, t = _edge_model(window)
+    toks = [0, 2, 3] * 70
+    for p in (3, 14, 15, 16, 31, 32, 47, 90):
+        toks[p] = 1
+    ref = R.forward(cfg, t, toks)
+    for wrong in (window - 1, window + 1):       # a window off by one token would show
+        if wrong >= 1:
+            other = dict(cfg, layers=[dict(cfg["layers"][0], mixer=dict(cfg["layers"][0]["mixer"], mask={"size": wrong}))])
+            assert (R.forward(other, t, toks) - ref).abs().max() > 0.1
+    engine, _ = build(cfg, dtype=dt, tensors=t, max_tokens=256, max_seqs=2)
+    close(whole(engine, "a", toks), ref, tol)
+    got = [engine.step([("b", toks[:61], list(range(61)))])]
+    for p in range(61, 200):
+        got.append(engine.step([("b", [toks[p]], [0])]))
+    engine.finish("b")
+    close(torch.cat(got).cpu(), ref[:200], tol)
+
+
+def test_one_far_key_among_hundreds_inside_a_long_window_bf16():
+    cfg, t = _edge_model(700)
+    toks = [0, 2, 3, 2, 0] * 160
+    toks[37] = 1
+    ref = R.forward(cfg, t, toks)
+    assert (ref[736] - ref[737]).abs().max() > 0.1           # 737 no longer sees it
+    engine, _ = build(cfg, dtype=torch.bfloat16, tensors=t, max_tokens=1024, max_seqs=1)
+    want = [36, 37, 300, 735, 736, 737, 738, 799]
+    close(whole(engine, "a", toks, want), ref[want], 0.03)
+
+
+# ---- the model through the engine ----------------------------------------------------------------------------------
+ALL = pytest.mark.parametrize("cfg", [CFG_A, CFG_B, CFG_C, CFG_D], ids=["A", "B", "C", "D"])
+AB = pytest.mark.parametrize("cfg", [CFG_A, CFG_B], ids=["A", "B"])
+
+
+@ALL
+def test_whole_prompt_fp32(cfg):
+    engine, tensors = build(cfg)
+    toks = tokens(90, cfg["vocab"], 11)
+    layers = []
+    ref = R.forward(cfg, tensors, toks, trace=layers)
+    engine.layer_trace = []
+    got = whole(engine, "a", toks)
+    for mine, theirs in zip(engine.layer_trace, layers):                    # the residual after every layer
+        close(mine.cpu(), theirs, 5e-5)
+    engine.layer_trace = None
+    close(got, ref, 5e-5)
+    one = tokens(1, cfg["vocab"], 12)                                       # the first token alone
+    close(whole(engine, "b", one), R.forward(cfg, tensors, one), 5e-5)
+
+
+@ALL
+def test_whole_prompt_bf16(cfg):
+    engine, tensors = build(cfg, dtype=torch.bfloat16)
+    toks = tokens(70, cfg["vocab"], 13)
+    rounding_close(whole(engine, "a", toks), R.forward(cfg, tensors, toks))
+
+
+@ALL
+def test_prefill_then_long_decode_matches_the_whole_prompt(cfg):
+    engine, tensors = build(cfg)
+    toks = tokens(120, cfg["vocab"], 14)
+    ref = R.forward(cfg, tensors, toks)
+    got = [engine.step([("a", toks[:30], list(range(30)))])]
+    for t in range(30, len(toks)):                               # 90 decoded tokens: the windows pass over them
+        got.append(engine.step([("a", [toks[t]], [0])]))
+    engine.finish("a")
+    close(torch.cat(got).cpu(), ref, 5e-5)
+    got = [engine.step([("b", [t], [0])]) for t in toks[:40]]    # decoding from the very first token, in a used slot
+    engine.finish("b")
+    close(torch.cat(got).cpu(), ref[:40], 5e-5)
+
+
+@AB
+def test_portions_of_any_size_down_to_two_tokens(cfg):
+    engine, tensors = build(cfg)
+    toks = tokens(131, cfg["vocab"], 15)
+    ref = R.forward(cfg, tensors, toks)
+    for cuts in ([2, 2, 13, 3, 16, 17, 2, 31, 33, 2, 1, 9], [64, 2, 65], [15, 1, 16, 1, 31, 1, 2, 64], [8, 1, 9, 1, 10, 102]):
+        got, at = [], 0
+        for c in cuts:
+            c = min(c, len(toks) - at)
+            got.append(engine.step([("a", toks[at:at + c], list(range(c)))]))
+            at += c
+        engine.finish("a")
+        close(torch.cat(got).cpu(), ref[:at], 5e-5)
+
+
+@AB
+def test_mixed_batches_match_each_request_alone_and_reuse_pages_and_slots(cfg):
+    engine, tensors = build(cfg, max_tokens=256, max_seqs=3)
+    prompts = {r: tokens(n, cfg["vocab"], 20 + i) for i, (r, n) in enumerate((("a", 70), ("b", 33), ("c", 5), ("d", 90), ("e", 48)))}
+    ref = {r: R.forward(cfg, tensors, t) for r, t in prompts.items()}
+    at = {r: 0 for r in prompts}
+    got = {r: [] for r in prompts}
+
+    def feed(plan):
+        out = engine.step([(r, prompts[r][at[r]:at[r] + c], list(range(c))) for r, c in plan])
+        o = 0
+        for r, c in plan:
+            got[r].append(out[o:o + c])
+            o, at[r] = o + c, at[r] + c
+            if at[r] == len(prompts[r]):
+                engine.finish(r)
+
+    feed([("a", 40), ("b", 2), ("c", 5)])                        # c ends: its slot and page are free again
+    feed([("a", 1), ("b", 30), ("d", 17)])                       # d takes c's slot (and must not read c's state)
+    feed([("b", 1), ("d", 2), ("a", 1)])                         # b ends
+    feed([("e", 1), ("a", 1), ("d", 1)])                         # e starts with a single token in b's slot
+    feed([("a", 1), ("e", 30), ("d", 1)])
+    feed([("d", 69), ("a", 26), ("e", 2)])                       # a and d end
+    feed([("e", 15)])
+    for r in prompts:
+        assert at[r] == len(prompts[r])
+        close(torch.cat(got[r]).cpu(), ref[r], 5e-5)
+    assert engine.free_slots == 3 and engine.free_blocks == 256 // 16
+
+
+@ALL
+def test_logits_do_not_depend_on_the_batch_or_the_cut_beyond_rounding_bf16(cfg):
+    engine, _ = build(cfg, dtype=torch.bfloat16)
+    a, b = tokens(80, cfg["vocab"], 31), tokens(37, cfg["vocab"], 32)
+    alone = whole(engine, "a", a)
+    out = engine.step([("b", b[:20], []), ("a", a[:50], list(range(50)))])
+    out2 = engine.step([("a", a[50:], list(range(30))), ("b", b[20:], [])])
+    engine.release()
+    rounding_close(torch.cat([out, out2]).cpu(), alone)
+
+
+def test_long_prompt_whole_in_portions_and_decoded_bf16_against_fp32():
+    """600 tokens through the tensor-core kernels: the whole prompt, portions beside another request, and single
+    tokens agree with the fp32 engine within 16-bit rounding."""
+    cfg = CFG_B
+    e32, _ = build(cfg, max_tokens=1024, max_seqs=2)
+    e16, _ = build(cfg, dtype=torch.bfloat16, max_tokens=1024, max_seqs=2)
+    toks = tokens(600, cfg["vocab"], 16)
+    want = [0, 100, 255, 256, 300, 400, 511, 512, 550, 590, 599]
+    ref = whole(e32, "a", toks, want)
+    rounding_close(whole(e16, "a", toks, want), ref)
+    got = [e16.step([("b", toks[:100], [0])]), e16.step([("b", toks[100:590], [0, 155, 156, 200, 300, 411, 412, 450]), ("c", toks[:3], [])])]
+    got += [e16.step([("b", [t], [0] if i in (0, 9) else [])]) for i, t in enumerate(toks[590:])]
+    e16.release()
+    rounding_close(torch.cat([g for g in got if g is not None]).cpu(), ref)
+
+
+def test_greedy_generation_through_the_scheduler():
+    cfg = CFG_B
+    engine, tensors = build(cfg, max_tokens=256, max_seqs=2)
+    prompts = [tokens(n, cfg["vocab"], 40 + i) for i, n in enumerate((9, 30, 3))]     # three requests, two slots
+    out = engine.generate(prompts, max_new_tokens=6, prefill_chunk=7, token_budget=12)
+    for p, o in zip(prompts, out):
+        want = R.greedy(cfg, tensors, p, 6)
+        # a near-tie may flip a token in fp32; up to the first difference the texts must agree and it must be a near-tie
+        for k, (x, y) in enumerate(zip(o, want)):
+            if x != y:
+                lg = R.forward(cfg, tensors, p + want[:k])[-1]
+                assert abs(lg[x] - lg[y]) < 1e-4
+                break
+    assert engine.free_slots == 2
+
+
+def test_registry_serves_a_checkpoint_folder(tmp_path):
+    import json
+
+    from dgi_b200 import model_registry, zuderax_layer as Z
+    from dgi_b200.ragged_engine import RaggedStepEngine
+    from dgi_b200.safetensors_io import write_safetensors
+
+    cfg = Z.ZuderaxConfig.from_dict(CFG_A)
+    tensors = Z.random_checkpoint(cfg, seed=5)
+    (tmp_path / "config.json").write_text(json.dumps(CFG_A))
+    write_safetensors(str(tmp_path / "model.safetensors"), tensors)
+    arch, _, shards = model_registry.load_model_dir(str(tmp_path), device=DEV, dtype=torch.float32)
+    assert arch.name == "Zuderax" and arch.engine == "ragged"
+    engine = RaggedStepEngine(shards, max_tokens=128, max_seqs=1)
+    toks = tokens(20, CFG_A["vocab"], 50)
+    close(whole(engine, "a", toks), R.forward(CFG_A, tensors, toks), 5e-5)
+
+
+def test_shards_cut_between_a_layer_and_the_layer_that_runs_its_weights():
+    from dgi_b200 import zuderax_layer as Z
+    from dgi_b200.ragged_engine import RaggedStepEngine
+
+    cfg = Z.ZuderaxConfig.from_dict(CFG_A)
+    tensors = Z.random_checkpoint(cfg, seed=6)
+    shards = Z.build_shards(cfg, tensors, [(0, 2), (2, 4), (4, 8)], DEV, torch.float32)
+    engine = RaggedStepEngine(shards, max_tokens=128, max_seqs=2)
+    toks = tokens(45, CFG_A["vocab"], 51)
+    ref = R.forward(CFG_A, tensors, toks)
+    got = [engine.step([("a", toks[:20], list(range(20)))]), engine.step([("a", toks[20:], list(range(25)))])]
+    close(torch.cat(got).cpu(), ref, 5e-5)
+    same = Z.build_shards(cfg, tensors, [(0, 8)], DEV, torch.float32)[0].layers
+    assert same[3].mixer is same[1].mixer and same[4].mlp is same[0].mlp and same[6].mixer is not same[1].mixer
