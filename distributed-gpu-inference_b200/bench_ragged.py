@@ -18,6 +18,11 @@ whose layers alternate attention and recurrence, again with every kernel of both
 key part and differential layers in turn, routed experts in every layer) beside a Fibirax model of equal width, depth,
 head layout and expert sizes (its closest relative here: post-norm sublayers that read the residual itself, windowed sink
 attention on the same tensor-core kernel, softmax routing over the same dispatch).
+
+``bench.py --compare zuderax``: the same two steps for the Zuderax model class (latent, matrix-memory and state-space layers,
+routed experts with a shared expert in every layer) beside the two models that have its like kernels, at equal width, depth,
+head layout and expert sizes: Fibirax (a decayed outer-product state per head in every layer, grouped routing, a shared
+expert) and Vatazen (the same latent attention).
 """
 from __future__ import annotations
 
@@ -599,6 +604,153 @@ def _vatazen_kernel_table(s, ev_prompt, ev_decode, B, Pn, Bd, ctx, hbm, tf) -> D
             "router_logits": (n_tok * W * 4, 0),
             "gather_rows": (n_tok * top * W * 4, 0),
             "weighted_expert_combine": (n_tok * top * W * 2 + n_tok * W * (4 + 4), 0),
+        }
+        for name, ts in by.items():
+            t = statistics.mean(ts)
+            entry = {"us": round(t * 1e6, 1), "calls": len(ts)}
+            if name in floors:
+                nbytes, flops = floors[name]
+                floor = max(nbytes / hbm, flops / tf)
+                entry["of_floor"] = round(floor / t, 3)
+                entry["bound"] = "math" if flops / tf > nbytes / hbm else "memory"
+            out.setdefault(phase, {})[name] = entry
+    return out
+
+
+# ---- Zuderax beside Fibirax and Vatazen ------------------------------------------------------------------------------
+ZUDERAX_STATE, ZUDERAX_VDIM, ZUDERAX_CONV = 128, 64, 4
+ZUDERAX_KINDS = ("latent_attention", "mlstm", "mamba2", "mlstm")     # one per layer
+
+
+def zuderax_config(s: Dict[str, int]) -> Dict[str, Any]:
+    """Matrix-memory layers take the size's recurrent heads as they are; state-space layers split the same inner width into
+    heads of 64 over a state of 128, one B / C group per 16 heads."""
+    lat = {"heads": s["heads"], "dim": s["dk"], "rot_dim": VATAZEN_ROT, "vdim": s["dv"], "kv_rank": VATAZEN_RANK,
+           "scale": 1.0 / math.sqrt(s["dk"] + VATAZEN_ROT), "mask": {"size": VATAZEN_WINDOW},
+           "rot": {"base": 10000.0, "dims": VATAZEN_ROT}}
+    mem = {"heads": s["rheads"], "dim": s["rdk"], "vdim": s["rdv"], "gate_cap": 15.0}
+    heads = s["rheads"] * s["rdv"] // ZUDERAX_VDIM
+    ssm = {"heads": heads, "vdim": ZUDERAX_VDIM, "state": ZUDERAX_STATE, "groups": heads // 16, "conv": ZUDERAX_CONV,
+           "norm_groups": heads // 16}
+    mixers = {"latent_attention": lat, "mlstm": mem, "mamba2": ssm}
+    mlp = {"kind": "moe", "expert": {"ff": s["eff"]}, "shared": {"ff": s["eff"]},
+           "router": {"experts": s["experts"], "top": s["top"], "scale": 2.0, "groups": {"count": 2, "keep": 1}}}
+    return {"architecture": "Zuderax", "width": s["width"], "vocab": VOCAB, "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+            "layers": [{"type": kind, "mixer": mixers[kind], "mlp": mlp} for kind in ZUDERAX_KINDS]}
+
+
+def _measure_ragged(mod, cfg, table, s, B, Pn, Bd, ctx, steps, warmup, prompts, hbm, tf):
+    """``(prompt tokens/s, decode tokens/s, kernel table)`` of a model class on the ragged step engine."""
+    from . import mixer_ops
+    from .ragged_engine import RaggedStepEngine
+
+    shards = mod.build_shards(cfg, mod.random_checkpoint(cfg, seed=0), [(0, LAYERS)], "cuda:0", torch.bfloat16)
+    eng = RaggedStepEngine(shards, max_tokens=Bd * (ctx + 64), max_seqs=Bd, fp32_logits=False)
+
+    def prompt_step():
+        eng.step([(i, prompts[i][:Pn], [Pn - 1]) for i in range(B)])
+        for i in range(B):
+            eng.finish(i)
+
+    def traced(fn):
+        mixer_ops.EVENTS = []
+        fn()
+        torch.cuda.synchronize()
+        events, mixer_ops.EVENTS = mixer_ops.EVENTS, None
+        return events
+
+    prefill = round(B * Pn / _time_steps(prompt_step, steps, warmup) * 1e3)
+    ev_prompt = traced(prompt_step)
+    for i in range(0, Bd, B):
+        eng.step([(j, prompts[j], []) for j in range(i, i + B)])
+
+    def decode_step():
+        eng.step([(j, [1], [0]) for j in range(Bd)])
+
+    n_dec = min(steps, 32)
+    decode = round(Bd / _time_steps(decode_step, n_dec, warmup) * 1e3)
+    ev_decode = traced(decode_step)
+    eng.release()
+    return prefill, decode, table(s, ev_prompt, ev_decode, B, Pn, Bd, ctx + warmup + n_dec, hbm, tf)
+
+
+def run_zuderax(args, measured_peaks, ClockSampler) -> None:
+    from . import fibirax_layer as Fx
+    from . import vatazen_layer as Vz
+    from . import zuderax_layer as Z
+
+    peaks, how = measured_peaks()
+    hbm, tf = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    steps, warmup = max(3, args.steps), max(3, args.warmup)
+    B, Pn, ctx, Bd = 8, 2048, 2048, 64
+    g = torch.Generator().manual_seed(0)
+    sampler = ClockSampler(0)
+    sampler.start()
+    report: Dict[str, Any] = {}
+    for name, s in SIZES.items():
+        if args.compare_sizes and name not in args.compare_sizes.split(","):
+            continue
+        row: Dict[str, Any] = {}
+        prompts = torch.randint(0, VOCAB, (Bd, ctx), generator=g).tolist()
+        for label, mod, cfg, table in (
+                ("zuderax", Z, Z.ZuderaxConfig(zuderax_config(s)), _zuderax_kernel_table),
+                ("fibirax", Fx, Fx.FibiraxConfig(fibirax_config(s)), _fibirax_kernel_table),
+                ("vatazen", Vz, Vz.VatazenConfig(vatazen_config(s)), _vatazen_kernel_table)):
+            prefill, decode, kernels = _measure_ragged(mod, cfg, table, s, B, Pn, Bd, ctx, steps, warmup, prompts, hbm, tf)
+            row[label + "_prefill_tok_s"], row[label + "_decode_tok_s"], row[label + "_kernels"] = prefill, decode, kernels
+            torch.cuda.empty_cache()
+        row["inputs_exceed_l2"] = bool(Bd * s["rheads"] * s["rdk"] * s["rdv"] * 4 * LAYERS > 126e6)
+        report[name] = row
+    clocks = sampler.stop()
+    print(json.dumps({"bench": "zuderax_vs_fibirax_and_vatazen", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic",
+                      "layers": LAYERS, "prompt_step": f"{B} x {Pn} tokens", "decode_step": f"{Bd} sequences at {ctx}",
+                      "peaks": how, "sizes": report, "clocks": clocks}), flush=True)
+
+
+def _zuderax_kernel_table(s, ev_prompt, ev_decode, B, Pn, Bd, ctx, hbm, tf) -> Dict[str, Any]:
+    """Like ``_kernel_table`` for the Zuderax kernels.  Calls of the shared state kernels are listed per layer type (the
+    order of a step's layers is fixed), those of the SiLU GLU per feed-forward (routed, then shared)."""
+    out: Dict[str, Any] = {}
+    W, H, dv, top, eff = s["width"], s["heads"], s["dv"], s["top"], s["eff"]
+    r, dr = VATAZEN_RANK, VATAZEN_ROT
+    RH, rdk, rdv = s["rheads"], s["rdk"], s["rdv"]
+    inner = RH * rdv
+    MH, N = inner // ZUDERAX_VDIM, ZUDERAX_STATE
+    bc = 2 * (MH // 16) * N
+    recurrent = [k for k in ZUDERAX_KINDS if k != "latent_attention"]
+    for phase, events, n_tok, past in (("prompt", ev_prompt, B * Pn, 0), ("decode", ev_decode, Bd, ctx)):
+        by: Dict[str, List[float]] = {}
+        calls: Dict[str, int] = {}
+        for name, a, b in events:
+            i = calls[name] = calls.get(name, -1) + 1
+            if name in ("decay_scan", "decay_step"):
+                name += f"[{recurrent[i % len(recurrent)]}]"
+            if name == "silu_glu":
+                name += "[routed]" if i % 2 == 0 else "[shared]"
+            by.setdefault(name, []).append(a.elapsed_time(b) * 1e-3)
+        per_seq = n_tok // (B if phase == "prompt" else Bd)
+        n_seq = n_tok // per_seq
+        pairs = sum(min(past + t + 1, VATAZEN_WINDOW) for t in range(per_seq))
+        keys = min(past + per_seq, VATAZEN_WINDOW + per_seq)
+        attn = (n_seq * keys * (r + dr) * 2 + n_tok * H * (2 * r + dr) * 2, n_seq * H * 2 * (2 * r + dr) * pairs)
+        mem = (n_tok * RH * ((2 * rdk + rdv) * 2 + rdv * 4) + 2 * n_seq * RH * rdk * rdv * 4, 0)
+        ssm = (n_tok * (inner * 6 + bc * 2) + 2 * n_seq * inner * N * 4, 0)
+        floors = {
+            "residual_dyn_tanh": (n_tok * W * (4 + 4 + 2 + 2), 0),
+            "expert_combine_dyn_tanh": (n_tok * W * (top * 2 + 2 + 4 + 4 + 2), 0),
+            "latent_rotary_append": (n_tok * (H * dr + r + dr) * 4, 0),
+            "mixed_prompt_attention": attn,
+            "decay_scan[mlstm]": mem, "decay_step[mlstm]": mem,
+            "decay_scan[mamba2]": ssm, "decay_step[mamba2]": ssm,
+            "capped_gates": (n_tok * RH * (4 + 12), 0),
+            "step_sizes": (n_tok * MH * (2 + 8), 0),
+            "normalized_head_out": (n_tok * inner * 8, 0),
+            "gated_part_norm": (n_tok * inner * 8, 0),
+            "causal_conv_silu": (n_tok * (inner + bc) * 4, 0),
+            "silu_glu[routed]": (n_tok * top * eff * 6, 0),
+            "silu_glu[shared]": (n_tok * eff * 6, 0),
+            "router_logits": (n_tok * W * 2, 0),
+            "gather_rows": (n_tok * top * W * 4, 0),
         }
         for name, ts in by.items():
             t = statistics.mean(ts)
