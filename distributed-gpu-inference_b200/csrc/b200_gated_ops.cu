@@ -252,11 +252,11 @@ gated_table_rows_kernel(T* __restrict__ out, const T* __restrict__ z, int64_t z_
 }
 
 // ---- router logits -------------------------------------------------------------------------------------------------
-// One CTA of four warps per token (or per few tokens), kRouterChunk experts at a time: thread t owns columns t, t + 128, ... (four at a time
-// when the width allows); partial sums meet in a butterfly per warp and the four warps' sums are added in warp order.
-// The order of every sum depends on the width alone, so a token's logits - and with them its experts - do not depend on
-// what else the step carries.
-constexpr int kRouterChunk = 8;
+// One CTA of four warps per TOK tokens, CH experts at a time: thread t owns columns t, t + 128, ... (four at a time when the
+// width allows); partial sums meet in a butterfly per warp and the four warps' sums are added in warp order.  The order of
+// every sum depends on the width alone, so a token's logits - and with them its experts - do not depend on what else the
+// step carries.  Experts past the last read the last one's weights and are dropped at the end: without a branch around them
+// the loads of all CH rows are in flight together.
 constexpr int kRouterThreads = 128;
 
 template <typename X>
@@ -270,61 +270,78 @@ __device__ __forceinline__ float4 row4(const X* p) {
   }
 }
 
-// TOK tokens per CTA share every weight that is read (steps of many tokens); a token's own sums do not see the others.
-template <typename X, bool VEC, int TOK>
+// TOK tokens per CTA share every weight that is read (steps of many tokens); a token's own sums do not see the others.  In
+// the butterfly's first log2(TOK) steps the two lanes of a pair keep half the tokens each: the same pairs are added in the
+// same order as in a full butterfly, with fewer shuffles.
+template <typename X, bool VEC, int TOK, int CH>
 __global__ void __launch_bounds__(kRouterThreads)
 router_logits_kernel(float* __restrict__ logits, const X* __restrict__ x, const float* __restrict__ w,
                      const float* __restrict__ bias, int64_t n_tok, int E, int W) {
-  __shared__ float part[kRouterThreads / 32][TOK][kRouterChunk];
+  static_assert((TOK & (TOK - 1)) == 0 && TOK <= 32 && TOK * CH <= kRouterThreads, "shape");
+  __shared__ float part[kRouterThreads / 32][TOK][CH];
   const int64_t n0 = static_cast<int64_t>(blockIdx.x) * TOK;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const X* xr[TOK];
 #pragma unroll
   for (int t = 0; t < TOK; ++t) xr[t] = x + (n0 + t < n_tok ? n0 + t : n0) * W;
-  for (int e0 = 0; e0 < E; e0 += kRouterChunk) {
-    float acc[TOK][kRouterChunk];
+  for (int e0 = 0; e0 < E; e0 += CH) {
+    float acc[TOK][CH];
+    const float* wr[CH];
+#pragma unroll
+    for (int j = 0; j < CH; ++j) wr[j] = w + static_cast<int64_t>(min(e0 + j, E - 1)) * W;
 #pragma unroll
     for (int t = 0; t < TOK; ++t)
 #pragma unroll
-      for (int j = 0; j < kRouterChunk; ++j) acc[t][j] = 0.f;
+      for (int j = 0; j < CH; ++j) acc[t][j] = 0.f;
     if (VEC) {
       for (int i = threadIdx.x * 4; i < W; i += kRouterThreads * 4) {
-        float4 xv[TOK];
+        float4 xv[TOK], wv[CH];
 #pragma unroll
         for (int t = 0; t < TOK; ++t) xv[t] = row4(xr[t] + i);
 #pragma unroll
-        for (int j = 0; j < kRouterChunk; ++j)
-          if (e0 + j < E) {
-            const float4 wv = *reinterpret_cast<const float4*>(w + static_cast<int64_t>(e0 + j) * W + i);
+        for (int j = 0; j < CH; ++j) wv[j] = *reinterpret_cast<const float4*>(wr[j] + i);
 #pragma unroll
-            for (int t = 0; t < TOK; ++t)
-              acc[t][j] = fmaf(xv[t].x, wv.x, fmaf(xv[t].y, wv.y, fmaf(xv[t].z, wv.z, fmaf(xv[t].w, wv.w, acc[t][j]))));
-          }
+        for (int j = 0; j < CH; ++j)
+#pragma unroll
+          for (int t = 0; t < TOK; ++t)
+            acc[t][j] = fmaf(xv[t].x, wv[j].x, fmaf(xv[t].y, wv[j].y, fmaf(xv[t].z, wv[j].z, fmaf(xv[t].w, wv[j].w, acc[t][j]))));
       }
     } else {
       for (int i = threadIdx.x; i < W; i += kRouterThreads) {
-        float xv[TOK];
+        float xv[TOK], wv[CH];
 #pragma unroll
         for (int t = 0; t < TOK; ++t) xv[t] = Cvt<X>::to_f32(xr[t][i]);
 #pragma unroll
-        for (int j = 0; j < kRouterChunk; ++j)
-          if (e0 + j < E) {
-            const float wv = w[static_cast<int64_t>(e0 + j) * W + i];
+        for (int j = 0; j < CH; ++j) wv[j] = wr[j][i];
 #pragma unroll
-            for (int t = 0; t < TOK; ++t) acc[t][j] = fmaf(xv[t], wv, acc[t][j]);
-          }
+        for (int j = 0; j < CH; ++j)
+#pragma unroll
+          for (int t = 0; t < TOK; ++t) acc[t][j] = fmaf(xv[t], wv[j], acc[t][j]);
       }
     }
+    int o = 16, tok = 0;
 #pragma unroll
-    for (int t = 0; t < TOK; ++t)
+    for (int half = TOK / 2; half > 0; half >>= 1, o >>= 1) {
+      const bool up = lane & o;
+      tok += up ? half : 0;
 #pragma unroll
-      for (int j = 0; j < kRouterChunk; ++j) {
-        const float s = warp_sum(acc[t][j]);
-        if (lane == 0) part[warp][t][j] = s;
-      }
+      for (int t = 0; t < half; ++t)
+#pragma unroll
+        for (int j = 0; j < CH; ++j) {
+          const float give = up ? acc[t][j] : acc[t + half][j];
+          acc[t][j] = (up ? acc[t + half][j] : acc[t][j]) + __shfl_xor_sync(0xffffffffu, give, o);
+        }
+    }
+#pragma unroll
+    for (; o > 0; o >>= 1)
+#pragma unroll
+      for (int j = 0; j < CH; ++j) acc[0][j] += __shfl_xor_sync(0xffffffffu, acc[0][j], o);
+    if ((lane & (32 / TOK - 1)) == 0)
+#pragma unroll
+      for (int j = 0; j < CH; ++j) part[warp][tok][j] = acc[0][j];
     __syncthreads();
-    if (threadIdx.x < TOK * kRouterChunk) {
-      const int t = threadIdx.x / kRouterChunk, j = threadIdx.x % kRouterChunk;
+    if (threadIdx.x < TOK * CH) {
+      const int t = threadIdx.x / CH, j = threadIdx.x % CH;
       if (e0 + j < E && n0 + t < n_tok) {
         float s = part[0][t][j];
 #pragma unroll
@@ -476,8 +493,9 @@ int b200_router_logits_ext(float* logits, const void* x, const float* w, const f
   if (n_tok < 0 || E <= 0 || width <= 0) return fail(B200_EINVAL, "b200_router_logits: bad sizes");
   if (n_tok == 0) return 0;
   if (!logits || !x || !w) return fail(B200_EINVAL, "b200_router_logits: null pointer");
-  constexpr int kTok = 4;
-  const bool many = n_tok >= 4 * kTok * kNumSMs;
+  constexpr int kTok = 8;
+  const bool many = n_tok >= 2 * kTok * kNumSMs;
+  const bool wide = (E + 11) / 12 * 12 < (E + 7) / 8 * 8;      // experts per pass: whichever leaves fewer idle
   const unsigned grid = static_cast<unsigned>(many ? (n_tok + kTok - 1) / kTok : n_tok);
   const bool vec = width % 4 == 0 && aligned16(x) && aligned16(w);
   return gated_by_dtype(dtype, "b200_router_logits", [&](auto* tag) {
@@ -486,10 +504,10 @@ int b200_router_logits_ext(float* logits, const void* x, const float* w, const f
       kern<<<grid, kRouterThreads, 0, static_cast<cudaStream_t>(stream)>>>(logits, static_cast<const X*>(x), w, bias, n_tok, E,
                                                                            width);
     };
-    if (vec && many) launch(router_logits_kernel<X, true, kTok>);
-    else if (vec) launch(router_logits_kernel<X, true, 1>);
-    else if (many) launch(router_logits_kernel<X, false, kTok>);
-    else launch(router_logits_kernel<X, false, 1>);
+    if (vec && many) wide ? launch(router_logits_kernel<X, true, kTok, 12>) : launch(router_logits_kernel<X, true, kTok, 8>);
+    else if (vec) wide ? launch(router_logits_kernel<X, true, 1, 12>) : launch(router_logits_kernel<X, true, 1, 8>);
+    else if (many) launch(router_logits_kernel<X, false, kTok, 8>);
+    else launch(router_logits_kernel<X, false, 1, 8>);
     return check_launch("b200_router_logits");
   });
 }

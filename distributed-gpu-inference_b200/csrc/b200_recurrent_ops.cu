@@ -568,7 +568,7 @@ decay_step_kernel(const StepArgs A) {
 // One warp per (token, head): o / (max(|nq|, exp(-m)) + floor), unit RMS, times w[h * dv + i], times sigmoid(gate).  When
 // m_state is given (steps of one token per sequence, row n = sequence n), the token's running maximum becomes the carried
 // one.
-template <typename T>
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256)
 normalized_head_out_kernel(T* __restrict__ out, int64_t out_stride, const float* __restrict__ o, const float* __restrict__ nq,
                            const float* __restrict__ m_seq, float floor_, const T* __restrict__ w, const T* __restrict__ gate,
@@ -579,44 +579,84 @@ normalized_head_out_kernel(T* __restrict__ out, int64_t out_stride, const float*
   const int lane = threadIdx.x & 31;
   const int64_t n = row / H;
   const int h = static_cast<int>(row - n * H);
-  const float m = m_seq[row];
-  const float den = fmaxf(fabsf(nq[row]), expf(-m)) + floor_;
   const float* x = o + row * dv;
-  float ss = 0.f;
-  for (int i = lane; i < dv; i += 32) {
-    const float y = x[i] / den;
-    ss = fmaf(y, y, ss);
-  }
-  const float inv = rsqrtf(warp_sum(ss) / static_cast<float>(dv) + eps);
   const T* gr = gate + n * gate_stride + static_cast<int64_t>(h) * dv;
   const T* wr = w + static_cast<int64_t>(h) * dv;
   T* dst = out + n * out_stride + static_cast<int64_t>(h) * dv;
-  for (int i = lane; i < dv; i += 32)
-    dst[i] = Cvt<T>::from_f32(x[i] / den * inv * Cvt<T>::to_f32(wr[i]) * sigmoid1(Cvt<T>::to_f32(gr[i])));
+  const float m = m_seq[row];
+  const float r = 1.0f / (fmaxf(fabsf(nq[row]), expf(-m)) + floor_);
+  float ss = 0.f;
+  if constexpr (VEC) {            // dv a multiple of 4, at most 512: the row stays in registers
+    float4 y[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int i = 4 * (lane + 32 * j);
+      y[j] = i < dv ? *reinterpret_cast<const float4*>(x + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+      y[j].x *= r;
+      y[j].y *= r;
+      y[j].z *= r;
+      y[j].w *= r;
+      ss = fmaf(y[j].x, y[j].x, fmaf(y[j].y, y[j].y, fmaf(y[j].z, y[j].z, fmaf(y[j].w, y[j].w, ss))));
+    }
+    const float inv = rsqrtf(warp_sum(ss) / static_cast<float>(dv) + eps);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int i = 4 * (lane + 32 * j);
+      if (i >= dv) break;
+      const float4 g = load4(gr + i), ww = load4(wr + i);
+      store4(dst + i, make_float4(y[j].x * inv * ww.x * sigmoid1(g.x), y[j].y * inv * ww.y * sigmoid1(g.y),
+                                  y[j].z * inv * ww.z * sigmoid1(g.z), y[j].w * inv * ww.w * sigmoid1(g.w)));
+    }
+  } else {
+    for (int i = lane; i < dv; i += 32) {
+      const float y = x[i] * r;
+      ss = fmaf(y, y, ss);
+    }
+    const float inv = rsqrtf(warp_sum(ss) / static_cast<float>(dv) + eps);
+    for (int i = lane; i < dv; i += 32)
+      dst[i] = Cvt<T>::from_f32(x[i] * r * inv * Cvt<T>::to_f32(wr[i]) * sigmoid1(Cvt<T>::to_f32(gr[i])));
+  }
   if (m_state != nullptr && lane == 0) m_state[static_cast<int64_t>(seqs[n].slot) * H + h] = m;
 }
 
-// One CTA per (token, part): y * silu(z) over the part's columns, unit RMS, times w.
-template <typename T>
+// One CTA per (token, part): y * silu(z) over the part's columns, unit RMS, times w.  V columns per access.
+template <typename T, int V>
 __global__ void __launch_bounds__(256)
 gated_part_norm_kernel(T* __restrict__ out, const float* __restrict__ y, const T* __restrict__ z, int64_t z_stride,
                        const T* __restrict__ w, float eps, int inner, int part) {
-  extern __shared__ float gn_row[];
+  extern __shared__ __align__(16) float gn_row[];
   __shared__ float red[32];
   const int64_t n = blockIdx.x;
   const int c0 = blockIdx.y * part;
   const float* yr = y + n * inner + c0;
   const T* zr = z + n * z_stride + c0;
   float ss = 0.f;
-  for (int i = threadIdx.x; i < part; i += blockDim.x) {
-    const float g = Cvt<T>::to_f32(zr[i]);
-    const float v = yr[i] * g * sigmoid1(g);
-    gn_row[i] = v;
-    ss = fmaf(v, v, ss);
+  for (int i = threadIdx.x * V; i < part; i += blockDim.x * V) {
+    if constexpr (V == 4) {
+      const float4 g = load4(zr + i);
+      float4 v = *reinterpret_cast<const float4*>(yr + i);
+      v.x *= g.x * sigmoid1(g.x);
+      v.y *= g.y * sigmoid1(g.y);
+      v.z *= g.z * sigmoid1(g.z);
+      v.w *= g.w * sigmoid1(g.w);
+      *reinterpret_cast<float4*>(gn_row + i) = v;
+      ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+    } else {
+      const float g = Cvt<T>::to_f32(zr[i]);
+      const float v = yr[i] * (g * sigmoid1(g));
+      gn_row[i] = v;
+      ss = fmaf(v, v, ss);
+    }
   }
   const float inv = rsqrtf(sum_over_block(ss, red) / static_cast<float>(part) + eps);
-  for (int i = threadIdx.x; i < part; i += blockDim.x)
-    out[n * inner + c0 + i] = Cvt<T>::from_f32(gn_row[i] * inv * Cvt<T>::to_f32(w[c0 + i]));
+  for (int i = threadIdx.x * V; i < part; i += blockDim.x * V) {     // every thread reads back what it wrote
+    if constexpr (V == 4) {
+      const float4 v = *reinterpret_cast<const float4*>(gn_row + i), ww = load4(w + c0 + i);
+      store4(out + n * inner + c0 + i, make_float4(v.x * inv * ww.x, v.y * inv * ww.y, v.z * inv * ww.z, v.w * inv * ww.w));
+    } else {
+      out[n * inner + c0 + i] = Cvt<T>::from_f32(gn_row[i] * inv * Cvt<T>::to_f32(w[c0 + i]));
+    }
+  }
 }
 
 }  // namespace
@@ -797,9 +837,15 @@ int b200_normalized_head_out(void* out, int64_t out_stride, const float* o, cons
   const int64_t rows = n_tok * H;
   return recurrent_by_dtype(dtype, "b200_normalized_head_out", [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
-    normalized_head_out_kernel<T><<<static_cast<unsigned>((rows + 7) / 8), 256, 0, static_cast<cudaStream_t>(stream)>>>(
-        static_cast<T*>(out), out_stride, o, nq, m_seq, floor_, static_cast<const T*>(w), static_cast<const T*>(gate),
-        gate_stride, eps, m_state, reinterpret_cast<const SeqSpan*>(seqs), rows, H, dv);
+    const bool vec = dv % 4 == 0 && dv <= 512 && gate_stride % 4 == 0 && out_stride % 4 == 0 && aligned16(o) && aligned16(w) &&
+                     aligned16(gate) && aligned16(out);
+    auto launch = [&](auto kern) {
+      kern<<<static_cast<unsigned>((rows + 7) / 8), 256, 0, static_cast<cudaStream_t>(stream)>>>(
+          static_cast<T*>(out), out_stride, o, nq, m_seq, floor_, static_cast<const T*>(w), static_cast<const T*>(gate),
+          gate_stride, eps, m_state, reinterpret_cast<const SeqSpan*>(seqs), rows, H, dv);
+    };
+    if (vec) launch(normalized_head_out_kernel<T, true>);
+    else launch(normalized_head_out_kernel<T, false>);
     return check_launch("b200_normalized_head_out");
   });
 }
@@ -812,13 +858,18 @@ int b200_gated_part_norm(void* out, const float* y, const void* z, int64_t z_str
   const int part = inner / parts;
   const size_t smem = sizeof(float) * static_cast<size_t>(part);
   if (smem > 200 * 1024 || parts > 65535) return fail(B200_ESHAPE, "b200_gated_part_norm: %d parts of %d", parts, part);
-  const int nt = part <= 64 ? 64 : (part <= 128 ? 128 : 256);
   return recurrent_by_dtype(dtype, "b200_gated_part_norm", [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
-    auto kern = gated_part_norm_kernel<T>;
-    if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
-    kern<<<dim3(static_cast<unsigned>(n_tok), parts), nt, smem, static_cast<cudaStream_t>(stream)>>>(
-        static_cast<T*>(out), y, static_cast<const T*>(z), z_stride, static_cast<const T*>(w), eps, inner, part);
+    const bool vec = part % 4 == 0 && z_stride % 4 == 0 && aligned16(y) && aligned16(z) && aligned16(w) && aligned16(out);
+    const int per = vec ? part / 4 : part;
+    const int nt = per <= 32 ? 32 : (per <= 64 ? 64 : (per <= 128 ? 128 : 256));
+    auto launch = [&](auto kern) {
+      if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+      kern<<<dim3(static_cast<unsigned>(n_tok), parts), nt, smem, static_cast<cudaStream_t>(stream)>>>(
+          static_cast<T*>(out), y, static_cast<const T*>(z), z_stride, static_cast<const T*>(w), eps, inner, part);
+    };
+    if (vec) launch(gated_part_norm_kernel<T, 4>);
+    else launch(gated_part_norm_kernel<T, 1>);
     return check_launch("b200_gated_part_norm");
   });
 }
