@@ -159,7 +159,7 @@ def test_silu_glu(dt, tol, ff):
 
 
 @DT
-@pytest.mark.parametrize("C,taps,bias", [(10, 4, True), (33, 1, True), (64, 4, True), (128, 3, False), (40, 8, True), (12, 11, True)])
+@pytest.mark.parametrize("C,taps,bias", [(10, 4, True), (33, 1, True), (64, 4, True), (128, 3, False), (40, 8, True), (12, 11, True), (64, 1, True), (40, 5, False)])
 def test_causal_convolution_with_bias_over_portions(dt, tol, C, taps, bias):
     from dgi_b200 import mixer_ops as M
 
