@@ -259,6 +259,47 @@ MIXER_SIGNATURES = {
     "b200_gated_part_norm": (
         c_int, [c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_float, c_int64, c_int, c_int, c_int,
                 c_void_p]),
+    # per-channel gates, weightless q/k norm, one decay per head, selective state spaces (csrc/b200_delta_chunk.cu,
+    # csrc/b200_selective_ops.cu)
+    "b200_mixed_paged_attn_ext2": (
+        c_int, [c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int, c_void_p, c_void_p,
+                c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_float, c_float, c_int, c_int, c_int,
+                c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "b200_mixed_prompt_attn_ext2": (
+        c_int, [c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int, c_void_p, c_void_p,
+                c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_float, c_int, c_int,
+                c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
+                c_int, c_void_p]),
+    "b200_mixed_prompt_attn_rows_supported": (c_int, [c_int, c_int, c_int, c_int, c_int]),
+    "b200_qknorm_rotary_append_ext2": (
+        c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_float, c_void_p,
+                c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                c_int64, c_int, c_void_p]),
+    "b200_delta_scan_ext": (
+        c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
+                c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p]),
+    "b200_delta_chunk_scan_supported": (
+        c_int, [c_int, c_int, c_int]),
+    "b200_delta_chunk_workspace": (
+        c_size_t, [c_int, c_int, c_int]),
+    "b200_delta_chunk_scan": (
+        c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
+                c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p,
+                c_int, c_void_p]),
+    "b200_delta_step": (
+        c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p,
+                c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_void_p]),
+    "b200_selective_scan": (
+        c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int64,
+                c_void_p, c_void_p, c_int64, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
+    "b200_selective_step": (
+        c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_void_p, c_int64,
+                c_void_p, c_void_p, c_int64, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
+    "b200_sandwich_residual": (
+        c_int, [c_void_p, c_void_p, c_int64, c_int, c_float, c_void_p, c_void_p, c_float, c_void_p, c_float, c_void_p,
+                c_int, c_int, c_int, c_void_p]),
+    "b200_gelu_glu": (
+        c_int, [c_void_p, c_void_p, c_int64, c_int, c_int, c_void_p]),
 }
 
 _lock = threading.Lock()
@@ -314,7 +355,7 @@ def _build_mixers() -> None:
         fcntl.flock(lock, fcntl.LOCK_EX)
         if os.path.exists(MIXER_LIB_PATH):
             return
-        proc = subprocess.run(["make", "-j6", "-C", csrc, "mixers"], stdout=subprocess.PIPE, stderr=subprocess.STDOUT)
+        proc = subprocess.run(["make", "-j8", "-C", csrc, "mixers"], stdout=subprocess.PIPE, stderr=subprocess.STDOUT)
         if proc.returncode != 0 or not os.path.exists(MIXER_LIB_PATH):
             raise B200LibraryError("building libb200_mixers.so failed:\n" + proc.stdout.decode(errors="replace")[-4000:])
 

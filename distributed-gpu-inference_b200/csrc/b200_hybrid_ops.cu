@@ -262,11 +262,17 @@ struct AttnArgs {
   int chunk = 0;   // > 0: a position sees only the keys of its own block of `chunk` positions (counted from 0)
   int v_row = 0;   // elements between value rows in v_pool (the value size unless the values are the first columns of wider rows)
   int v_div = 1;   // value head = key head / v_div (several key heads read one value head)
-  int row_heads = 0;   // tensor-core kernel, > 0: a tile is ONE token and its 16 rows are consecutive heads of `row_heads`
-                       // that share one kv head; H then counts groups of 16 heads
+  int row_heads = 0;   // tensor-core kernel, > 0: a tile is ONE token and its 16 rows are consecutive heads of the `row_heads`
+                       // that share a kv head; H then counts groups of 16 heads (or what is left of a kv head's)
   int out_f32 = 0;     // != 0: `out` is fp32 (same strides, in elements) whatever T is; plain outputs only (no turn back)
   int stage_q = 0;     // tensor-core kernel: a warp's 16 query rows are staged in shared memory once (always with row_heads)
+  int gate_dim = 0;    // 0: one gate per head (rows of H); the value size: one per output channel (rows of H * dv)
 };
+
+template <typename T>
+__device__ __forceinline__ float gate_at(const AttnArgs& A, const T* gate, int64_t n, int h, int c) {
+  return sigmoid_(Cvt<T>::to_f32(gate[n * A.gate_stride + (A.gate_dim ? h * A.gate_dim + c : h)]));
+}
 
 // first key a position sees (the kept first tokens of a window aside)
 __device__ __forceinline__ int first_visible(const AttnArgs& A, int p) {
@@ -463,7 +469,7 @@ mixed_paged_attn_kernel(const AttnArgs A) {
       const int hl = e / dv, c = e - hl * dv;
       if (h0 + hl >= H) continue;
       float y = res[e];
-      if (gate) y *= sigmoid_(Cvt<T>::to_f32(gate[static_cast<int64_t>(n) * A.gate_stride + h0 + hl]));
+      if (gate) y *= gate_at(A, gate, n, h0 + hl, c);
       if (A.out_f32) static_cast<float*>(A.out)[static_cast<int64_t>(n) * A.out_tok_stride + (h0 + hl) * A.out_head_stride + c] = y;
       else out[(h0 + hl) * A.out_head_stride + c] = Cvt<T>::from_f32(y);
     }
@@ -558,6 +564,10 @@ mixed_prompt_attn_kernel(const AttnArgs A, const int32_t* __restrict__ tiles, co
   float* raw = reinterpret_cast<float*>(stage0 + stages * stage_elems);         // [H][16][40]
   float* talk_s = raw + (mixed ? H * kTcRows * kTcRawStride : 0);                               // [HC][H]
   const int RH = EXT ? A.row_heads : 0;
+  // heads on the rows: group h of 16 rows starts at head `head0(h)` and holds `rows_of(h)` of its kv head's heads
+  const int PG = RH ? (RH + 15) / 16 : 1;
+  auto head0 = [&](int h) { return RH ? (h / PG) * RH + 16 * (h % PG) : h; };
+  auto rows_of = [&](int h) { return RH ? min(16, RH - 16 * (h % PG)) : cnt; };
   // a warp's 16 query rows staged once: few resident warps cannot hide the latency of re-reading them for every key tile
   // (heads on the rows: one warp per CTA; wide value layouts: one CTA per SM)
   const bool QS = EXT && A.stage_q;
@@ -570,10 +580,9 @@ mixed_prompt_attn_kernel(const AttnArgs A, const int32_t* __restrict__ tiles, co
       for (int e = lane; e < kTcRows * kch; e += 32) {
         const int r = e / kch, ch = e - r * kch;
         int4 v = make_int4(0, 0, 0, 0);
-        const bool ok = RH ? 16 * h + r < RH : r < cnt;
-        if (ok)
+        if (r < rows_of(h))
           v = *reinterpret_cast<const int4*>(static_cast<const T*>(A.q) +
-                                             (RH ? static_cast<int64_t>(row0) * A.q_tok_stride + (16 * h + r) * A.q_head_stride
+                                             (RH ? static_cast<int64_t>(row0) * A.q_tok_stride + (head0(h) + r) * A.q_head_stride
                                                  : static_cast<int64_t>(row0 + r) * A.q_tok_stride + h * A.q_head_stride) + ch * 8);
         *reinterpret_cast<int4*>(q_s + (hl * kTcRows + r) * ks + ch * 8) = v;
       }
@@ -615,7 +624,7 @@ mixed_prompt_attn_kernel(const AttnArgs A, const int32_t* __restrict__ tiles, co
     const T* qa = QS ? q_s + ((h - h0) * kTcRows + qr) * ks + qc
                      : qbase + static_cast<int64_t>(row0 + qr) * A.q_tok_stride + h * A.q_head_stride + qc;
     const T* qb = qa + 8 * (QS ? static_cast<int64_t>(ks) : A.q_tok_stride);
-    const int rows = RH ? min(16, RH - 16 * h) : cnt;
+    const int rows = rows_of(h);
     const bool va = qr < rows, vb = qr + 8 < rows;
     const T* kt = Ks + (h / rep - g_lo) * kTcKeys * ks + qr * ks + qc;
     for (int kk = 0; kk < dk; kk += 16) {
@@ -716,7 +725,7 @@ mixed_prompt_attn_kernel(const AttnArgs A, const int32_t* __restrict__ tiles, co
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         const int row = qr + 8 * half, p = RH ? p0 : p0 + row;
-        const bool row_ok = row < (RH ? min(16, RH - 16 * h) : cnt);
+        const bool row_ok = row < rows_of(h);
         const int lo_p = first_seen(p);
         float mx = -INFINITY;
 #pragma unroll
@@ -786,8 +795,8 @@ mixed_prompt_attn_kernel(const AttnArgs A, const int32_t* __restrict__ tiles, co
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         const int row = qr + 8 * half;
-        if (row >= (RH ? min(16, RH - 16 * h) : cnt)) continue;
-        float* dst = RH ? ws + ((static_cast<int64_t>(blockIdx.z) * n_tok + row0) * RH + 16 * h + row) * (DVP + 2)
+        if (row >= rows_of(h)) continue;
+        float* dst = RH ? ws + ((static_cast<int64_t>(blockIdx.z) * n_tok + row0) * (RH * G) + head0(h) + row) * (DVP + 2)
                         : ws + ((static_cast<int64_t>(blockIdx.z) * n_tok + row0 + row) * H + h) * (DVP + 2);
         if (qc == 0) {
           dst[0] = m_r[hw][half];
@@ -812,16 +821,17 @@ mixed_prompt_attn_kernel(const AttnArgs A, const int32_t* __restrict__ tiles, co
     for (int half = 0; half < 2; ++half) {
       const int row = qr + 8 * half;
       float f = 0.f;
-      if (row < (RH ? min(16, RH - 16 * h) : cnt)) {
+      if (row < rows_of(h)) {
         float m = m_r[hw][half], l = l_r[hw][half];
         if (A.sink) {
-          const float sk = A.sink[RH ? 16 * h + row : h], M = fmaxf(m, sk);
+          const float sk = A.sink[RH ? head0(h) + row : h], M = fmaxf(m, sk);
           l = l * expf(m - M) + expf(sk - M);
           f = expf(m - M) / l;
         } else {
           f = 1.0f / l;
         }
-        if (gate && !A.unrotate) f *= sigmoid_(Cvt<T>::to_f32(gate[static_cast<int64_t>(row0 + row) * A.gate_stride + h]));
+        if (gate && !A.unrotate && !(EXT && A.gate_dim))
+          f *= sigmoid_(Cvt<T>::to_f32(gate[static_cast<int64_t>(RH ? row0 : row0 + row) * A.gate_stride + (RH ? head0(h) + row : h)]));
       }
 #pragma unroll
       for (int nt = 0; nt < DV8; ++nt) {
@@ -833,13 +843,18 @@ mixed_prompt_attn_kernel(const AttnArgs A, const int32_t* __restrict__ tiles, co
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         const int row = qr + 8 * half;
-        if (row >= (RH ? min(16, RH - 16 * h) : cnt)) continue;
-        T* orow = RH ? outp + static_cast<int64_t>(row0) * A.out_tok_stride + (16 * h + row) * A.out_head_stride
+        if (row >= rows_of(h)) continue;
+        T* orow = RH ? outp + static_cast<int64_t>(row0) * A.out_tok_stride + (head0(h) + row) * A.out_head_stride
                      : outp + static_cast<int64_t>(row0 + row) * A.out_tok_stride + h * A.out_head_stride;
 #pragma unroll
         for (int nt = 0; nt < DV8; ++nt) {
           const int c = nt * 8 + qc;
           if (c >= dv) continue;
+          if (EXT && gate && A.gate_dim) {
+            const int64_t tok = RH ? row0 : row0 + row;
+            O[hw][nt][2 * half] *= gate_at(A, gate, tok, RH ? head0(h) + row : h, c);
+            O[hw][nt][2 * half + 1] *= gate_at(A, gate, tok, RH ? head0(h) + row : h, c + 1);
+          }
           if (EXT && A.out_f32)
             *reinterpret_cast<float2*>(static_cast<float*>(A.out) + (orow - outp) + c) = make_float2(O[hw][nt][2 * half], O[hw][nt][2 * half + 1]);
           else
@@ -928,7 +943,7 @@ attn_split_combine_kernel(const AttnArgs A, const float* __restrict__ ws, int n_
     for (int e = threadIdx.x; e < H * dv; e += blockDim.x) {
       const int h = e / dv, c = e - h * dv;
       float y = res[e];
-      if (gate) y *= sigmoid_(Cvt<T>::to_f32(gate[static_cast<int64_t>(n) * A.gate_stride + h]));
+      if (gate) y *= gate_at(A, gate, n, h, c);
       if (A.out_f32) static_cast<float*>(A.out)[static_cast<int64_t>(n) * A.out_tok_stride + h * A.out_head_stride + c] = y;
       else out[h * A.out_head_stride + c] = Cvt<T>::from_f32(y);
     }
@@ -1083,7 +1098,7 @@ causal_conv_silu_kernel(T* __restrict__ out, int64_t out_stride, const T* __rest
 // column in registers for the whole portion.  Eight tokens (fewer for the widest keys) are staged at a time, double buffered (the raw loads of
 // the next eight are issued before the current eight are computed): their activated q and k (unit length per head, q
 // also scaled), the decays g = exp(-exp(A_log) softplus(a + dt_bias)), the write strength sigmoid(b) and the CTA's
-// value columns.  Per token: S <- g S and d = S^T k in one pass, u = beta (v - d), then S <- S + k u and
+// value columns (the decays as g - 1, so that one just below 1 is not rounded alike token after token).  Per token: S <- g S and d = S^T k in one pass, u = beta (v - d), then S <- S + k u and
 // o = S^T q in a second pass; the four lanes' partial sums meet in two shuffles.
 constexpr int kDeltaNT = 128;
 constexpr int kDeltaCols = kDeltaNT / 4;
@@ -1096,6 +1111,7 @@ struct DeltaArgs {
   const void* dt_bias; const void* a_log;
   float* state; const SeqSpan* seqs;
   int H, G, dk, dv; float unit_eps, q_scale;
+  int per_channel;   // 1: a decay logit and a bias per key channel, 0: one of each per head
 };
 
 __host__ __device__ constexpr int delta_chunk(int dk_padded) { return dk_padded >= 256 ? 2 : (dk_padded >= 128 ? 4 : 8); }
@@ -1149,7 +1165,7 @@ delta_scan_kernel(const DeltaArgs A) {
           if (i < dk) {
             if (which == 0) rawv[u] = qp[tok * A.in_stride + gq * dk + i];
             else if (which == 1) rawv[u] = kp[tok * A.in_stride + gq * dk + i];
-            else rawv[u] = ap[tok * A.a_stride + h * dk + i];
+            else rawv[u] = ap[tok * A.a_stride + (A.per_channel ? h * dk + i : h)];
           }
         } else if (sl < 3 * DK + kDeltaCols) {
           if (sl - 3 * DK < ncol) rawv[u] = vp[tok * A.in_stride + h * dv + col0 + sl - 3 * DK];
@@ -1169,7 +1185,7 @@ delta_scan_kernel(const DeltaArgs A) {
         if (sl >= 2 * DK && sl < 3 * DK) {
           const int s2 = sl - 2 * DK;
           const int i = 4 * (s2 % RW4) + s2 / RW4;
-          val = i < dk ? expf(-a_rate * softplus_(val + Cvt<T>::to_f32(dtb[h * dk + i]))) : 0.f;
+          val = i < dk ? expm1f(-a_rate * softplus_(val + Cvt<T>::to_f32(dtb[A.per_channel ? h * dk + i : h]))) : 0.f;
         } else if (sl == 3 * DK + kDeltaCols) {
           val = sigmoid_(val);
         }
@@ -1215,13 +1231,13 @@ delta_scan_kernel(const DeltaArgs A) {
       for (int kk = 0; kk < RW4; kk += 4) {
         const float4 g4 = *reinterpret_cast<const float4*>(gr + kk);
         const float4 k4 = *reinterpret_cast<const float4*>(kr + kk);
-        S[kk] *= g4.x;
+        S[kk] = fmaf(g4.x, S[kk], S[kk]);
         d0 = fmaf(S[kk], k4.x, d0);
-        S[kk + 1] *= g4.y;
+        S[kk + 1] = fmaf(g4.y, S[kk + 1], S[kk + 1]);
         d1 = fmaf(S[kk + 1], k4.y, d1);
-        S[kk + 2] *= g4.z;
+        S[kk + 2] = fmaf(g4.z, S[kk + 2], S[kk + 2]);
         d0 = fmaf(S[kk + 2], k4.z, d0);
-        S[kk + 3] *= g4.w;
+        S[kk + 3] = fmaf(g4.w, S[kk + 3], S[kk + 3]);
         d1 = fmaf(S[kk + 3], k4.w, d1);
       }
       float d = d0 + d1;
@@ -1395,6 +1411,20 @@ int b200_mixed_paged_attn_ext(void* out, int64_t out_tok_stride, int64_t out_hea
                               const float* sink, float scale, float softcap, int window, int keep_first, int chunk,
                               int unrotate, int interleaved, float rot_base, int H, int G, int dk, int dv, int v_row,
                               int v_div, int out_f32, int block_size, int dtype, void* stream) {
+  return b200_mixed_paged_attn_ext2(out, out_tok_stride, out_head_stride, q, q_tok_stride, q_head_stride, gate, gate_stride,
+                                    0, k_pool, v_pool, block_tables, table_stride, tok_row, tok_pos, n_tok, talk, sink, scale,
+                                    softcap, window, keep_first, chunk, unrotate, interleaved, rot_base, H, G, dk, dv, v_row,
+                                    v_div, out_f32, block_size, dtype, stream);
+}
+
+int b200_mixed_paged_attn_ext2(void* out, int64_t out_tok_stride, int64_t out_head_stride, const void* q,
+                               int64_t q_tok_stride, int64_t q_head_stride, const void* gate, int64_t gate_stride,
+                               int gate_per_channel, const void* k_pool, const void* v_pool, const int32_t* block_tables,
+                               int table_stride, const int32_t* tok_row, const int32_t* tok_pos, int n_tok,
+                               const float* talk, const float* sink, float scale, float softcap, int window, int keep_first,
+                               int chunk, int unrotate, int interleaved, float rot_base, int H, int G, int dk, int dv,
+                               int v_row, int v_div, int out_f32, int block_size, int dtype, void* stream) {
+  if (gate_per_channel && unrotate) return fail(B200_EINVAL, "b200_mixed_paged_attn: a gate per channel is not turned back");
   if (out_f32 && unrotate) return fail(B200_EINVAL, "b200_mixed_paged_attn: fp32 outputs are not turned back");
   if (n_tok < 0 || H <= 0 || G <= 0 || H % G || dk <= 0 || dv <= 0 || block_size <= 0 || chunk < 0 || v_row < dv ||
       v_div < 1 || G % v_div)
@@ -1405,7 +1435,8 @@ int b200_mixed_paged_attn_ext(void* out, int64_t out_tok_stride, int64_t out_hea
     return fail(B200_EINVAL, "b200_mixed_paged_attn: null pointer");
   AttnArgs A{out, out_tok_stride, out_head_stride, q, q_tok_stride, q_head_stride, gate, gate_stride, k_pool, v_pool,
              block_tables, table_stride, tok_row, tok_pos, talk, sink, scale, window, keep_first, unrotate, interleaved,
-             static_cast<double>(rot_base), H, G, dk, dv, block_size, softcap, chunk, v_row, v_div, 0, out_f32};
+             static_cast<double>(rot_base), H, G, dk, dv, block_size, softcap, chunk, v_row, v_div, 0, out_f32, 0,
+             gate_per_channel ? dv : 0};
   const int dvc = dv <= 64 ? 2 : (dv <= 128 ? 4 : (dv <= 256 ? 8 : 16));
   const int hp = dvc <= 4 ? 8 : (dvc == 8 ? 4 : 2);
   const int nhs = talk ? H : std::min(hp, H);
@@ -1432,6 +1463,11 @@ int b200_mixed_paged_attn_ext(void* out, int64_t out_tok_stride, int64_t out_hea
 int b200_mixed_prompt_attn_supported(int H, int G, int dk, int dv, int has_talk, int same_pool, int unrotate, int dtype) {
   if (H <= 0 || G <= 0) return 0;
   return tc_plan(H, G, dk, dv, has_talk != 0, same_pool != 0, unrotate != 0, dtype, nullptr) ? 1 : 0;
+}
+
+int b200_mixed_prompt_attn_rows_supported(int H, int G, int dk, int dv, int dtype) {
+  if (H <= 0 || G <= 0 || H % G) return 0;
+  return tc_plan(G * ((H / G + 15) / 16), G, dk, dv, false, false, false, dtype, nullptr, true) ? 1 : 0;
 }
 
 int b200_mixed_prompt_attn_splits(int n_tiles, int key_tiles, int H, int G, int dk, int dv, int has_talk, int same_pool,
@@ -1471,15 +1507,32 @@ int b200_mixed_prompt_attn_ext(void* out, int64_t out_tok_stride, int64_t out_he
                                const float* value_rot, int interleaved, int H, int G, int dk, int dv, int v_row, int v_div,
                                int heads_as_rows, int out_f32, int block_size, int n_splits, float* workspace, int dtype,
                                void* stream) {
+  if (heads_as_rows && (G != 1 || gate))
+    return fail(B200_EINVAL, "b200_mixed_prompt_attn: heads as rows need one kv head and no mixing, gate or value rotation");
+  return b200_mixed_prompt_attn_ext2(out, out_tok_stride, out_head_stride, q, q_tok_stride, q_head_stride, gate, gate_stride,
+                                     0, k_pool, v_pool, block_tables, table_stride, tiles, n_tiles, tok_pos, n_tok, talk,
+                                     sink, scale, softcap, window, keep_first, chunk, value_rot, interleaved, H, G, dk, dv,
+                                     v_row, v_div, heads_as_rows, out_f32, block_size, n_splits, workspace, dtype, stream);
+}
+
+int b200_mixed_prompt_attn_ext2(void* out, int64_t out_tok_stride, int64_t out_head_stride, const void* q,
+                                int64_t q_tok_stride, int64_t q_head_stride, const void* gate, int64_t gate_stride,
+                                int gate_per_channel, const void* k_pool, const void* v_pool, const int32_t* block_tables,
+                                int table_stride, const int32_t* tiles, int n_tiles, const int32_t* tok_pos, int n_tok,
+                                const float* talk, const float* sink, float scale, float softcap, int window,
+                                int keep_first, int chunk, const float* value_rot, int interleaved, int H, int G, int dk,
+                                int dv, int v_row, int v_div, int heads_as_rows, int out_f32, int block_size, int n_splits,
+                                float* workspace, int dtype, void* stream) {
+  if (gate_per_channel && value_rot) return fail(B200_EINVAL, "b200_mixed_prompt_attn: a gate per channel is not turned back");
   if (out_f32 && value_rot) return fail(B200_EINVAL, "b200_mixed_prompt_attn: fp32 outputs are not turned back");
   if (chunk < 0 || v_row < dv || v_row % 8 || v_div < 1 || G % v_div)
     return fail(B200_EINVAL, "b200_mixed_prompt_attn: bad mask or value layout");
-  if (heads_as_rows && (G != 1 || talk || gate || value_rot))
-    return fail(B200_EINVAL, "b200_mixed_prompt_attn: heads as rows need one kv head and no mixing, gate or value rotation");
+  if (heads_as_rows && (G <= 0 || H % G || v_div != 1 || talk || value_rot))
+    return fail(B200_EINVAL, "b200_mixed_prompt_attn: heads as rows allow no mixing, shared values or value rotation");
   if (heads_as_rows && (!aligned16(q) || ((q_tok_stride | q_head_stride) & 7)))
     return fail(B200_ESHAPE, "b200_mixed_prompt_attn: heads as rows need 16-byte aligned query rows");
   const int H_real = H;
-  if (heads_as_rows) H = (H + 15) / 16;      // the kernel's heads are groups of 16 rows
+  if (heads_as_rows) H = G * ((H / G + 15) / 16);      // the kernel's heads are groups of up to 16 rows of one kv head
   if (n_tiles < 0 || n_tok < 0 || H <= 0 || G <= 0 || H % G || dk <= 0 || dv <= 0 || block_size <= 0 || n_splits < 1 ||
       n_splits > 64)
     return fail(B200_EINVAL, "b200_mixed_prompt_attn: bad sizes");
@@ -1492,7 +1545,7 @@ int b200_mixed_prompt_attn_ext(void* out, int64_t out_tok_stride, int64_t out_he
   // query rows are staged where few warps are resident anyway: heads on the rows, and the widest value layout (one CTA
   // per SM by its registers) when its rows allow 16-byte reads
   const bool q_ok = aligned16(q) && !((q_tok_stride | q_head_stride) & 7);
-  const bool ext_call = chunk > 0 || v_div > 1 || v_row != dv || heads_as_rows || out_f32;
+  const bool ext_call = chunk > 0 || v_div > 1 || v_row != dv || heads_as_rows || out_f32 || gate_per_channel;
   bool stage_q = heads_as_rows || (ext_call && dv > 128 && q_ok);
   if (stage_q && !heads_as_rows && !tc_plan(H, G, dk, dv, talk != nullptr, k_pool == v_pool, value_rot != nullptr, dtype, &plan, true))
     stage_q = false;
@@ -1500,8 +1553,8 @@ int b200_mixed_prompt_attn_ext(void* out, int64_t out_tok_stride, int64_t out_he
     return fail(B200_ESHAPE, "b200_mixed_prompt_attn: sizes off the tensor-core grid (dk %d, dv %d)", dk, dv);
   AttnArgs A{out, out_tok_stride, out_head_stride, q, q_tok_stride, q_head_stride, gate, gate_stride, k_pool, v_pool,
              block_tables, table_stride, nullptr, tok_pos, talk, sink, scale, window, keep_first, value_rot != nullptr,
-             interleaved, 0.0, H, G, dk, dv, block_size, softcap, chunk, v_row, v_div, heads_as_rows ? H_real : 0,
-             out_f32, stage_q ? 1 : 0};
+             interleaved, 0.0, H, G, dk, dv, block_size, softcap, chunk, v_row, v_div, heads_as_rows ? H_real / G : 0,
+             out_f32, stage_q ? 1 : 0, gate_per_channel ? dv : 0};
   const dim3 grid(n_tiles, (H + kTcWarps * plan.hw - 1) / (kTcWarps * plan.hw), n_splits);
   return hybrid_by_dtype(dtype, "b200_mixed_prompt_attn", [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
@@ -1588,6 +1641,14 @@ int b200_delta_scan(float* o_raw, const void* q, const void* k, const void* v, i
                     int64_t beta_stride, const void* a_logit, int64_t a_stride, const void* dt_bias, const void* a_log,
                     float* state, const int32_t* seqs, int n_seqs, int H, int G, int dk, int dv, float unit_eps,
                     float q_scale, int dtype, void* stream) {
+  return b200_delta_scan_ext(o_raw, q, k, v, in_stride, beta_logit, beta_stride, a_logit, a_stride, dt_bias, a_log, 1, state,
+                             seqs, n_seqs, H, G, dk, dv, unit_eps, q_scale, dtype, stream);
+}
+
+int b200_delta_scan_ext(float* o_raw, const void* q, const void* k, const void* v, int64_t in_stride, const void* beta_logit,
+                        int64_t beta_stride, const void* a_logit, int64_t a_stride, const void* dt_bias, const void* a_log,
+                        int per_channel, float* state, const int32_t* seqs, int n_seqs, int H, int G, int dk, int dv,
+                        float unit_eps, float q_scale, int dtype, void* stream) {
   if (n_seqs < 0 || H <= 0 || G <= 0 || H % G || dk <= 0 || dv <= 0) return fail(B200_EINVAL, "b200_delta_scan: bad sizes");
   if (dk > 256) return fail(B200_ESHAPE, "b200_delta_scan: key size %d beyond 256", dk);
   if (n_seqs == 0) return 0;
@@ -1597,7 +1658,7 @@ int b200_delta_scan(float* o_raw, const void* q, const void* k, const void* v, i
   const size_t smem = sizeof(float) * 2 * delta_chunk(dkt) * (3 * static_cast<size_t>(dkt) + kDeltaCols + 4);
   const dim3 grid(n_seqs, H, (dv + kDeltaCols - 1) / kDeltaCols);
   DeltaArgs A{o_raw, q, k, v, in_stride, beta_logit, beta_stride, a_logit, a_stride, dt_bias, a_log, state,
-              reinterpret_cast<const SeqSpan*>(seqs), H, G, dk, dv, unit_eps, q_scale};
+              reinterpret_cast<const SeqSpan*>(seqs), H, G, dk, dv, unit_eps, q_scale, per_channel};
   return hybrid_by_dtype(dtype, "b200_delta_scan", [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
     auto s = static_cast<cudaStream_t>(stream);

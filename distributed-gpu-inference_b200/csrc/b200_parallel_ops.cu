@@ -60,7 +60,7 @@ template <typename T>
 __global__ void __launch_bounds__(kQkWarps * 32)
 qknorm_rotary_append_kernel(T* __restrict__ q, int64_t q_stride, const T* __restrict__ k, int64_t k_stride,
                             const T* __restrict__ v, int64_t v_stride, const T* __restrict__ qw, const T* __restrict__ kw,
-                            float eps, const double* __restrict__ freqs, int rot_dims, int interleaved,
+                            int unit_norm, float eps, const double* __restrict__ freqs, int rot_dims, int interleaved,
                             T* __restrict__ k_pool, T* __restrict__ v_pool, const int64_t* __restrict__ slot_mapping,
                             const int32_t* __restrict__ tok_pos, int H, int G, int Gv, int dk, int dv, int block_size) {
   extern __shared__ float qk_sm[];     // cos[rh] sin[rh] slab[warps][dk]
@@ -93,9 +93,9 @@ qknorm_rotary_append_kernel(T* __restrict__ q, int64_t q_stride, const T* __rest
       slab[i] = x;
       ss = fmaf(x, x, ss);
     }
-    if (w != nullptr) {
+    if (w != nullptr || unit_norm) {   // a rotation keeps the row's length: without a weight, before it is after it
       const float inv = rsqrtf(warp_sum(ss) / static_cast<float>(dk) + eps);
-      for (int i = lane; i < dk; i += 32) slab[i] = slab[i] * inv * Cvt<T>::to_f32(w[i]);
+      for (int i = lane; i < dk; i += 32) slab[i] = slab[i] * inv * (w ? Cvt<T>::to_f32(w[i]) : 1.0f);
     }
     __syncwarp();
     for (int i = lane; i < rh; i += 32) {
@@ -595,6 +595,16 @@ int b200_qknorm_rotary_append_ext(void* q, int64_t q_stride, const void* k, int6
                                   int rot_dims, int interleaved, void* k_pool, void* v_pool, const int64_t* slot_mapping,
                                   const int32_t* tok_pos, int n_tok, int H, int G, int Gv, int dk, int dv, int block_size,
                                   int64_t max_blocks, int dtype, void* stream) {
+  return b200_qknorm_rotary_append_ext2(q, q_stride, k, k_stride, v, v_stride, q_norm, k_norm, 0, eps, freqs, rot_dims,
+                                        interleaved, k_pool, v_pool, slot_mapping, tok_pos, n_tok, H, G, Gv, dk, dv,
+                                        block_size, max_blocks, dtype, stream);
+}
+
+int b200_qknorm_rotary_append_ext2(void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v,
+                                   int64_t v_stride, const void* q_norm, const void* k_norm, int unit_norm, float eps,
+                                   const double* freqs, int rot_dims, int interleaved, void* k_pool, void* v_pool,
+                                   const int64_t* slot_mapping, const int32_t* tok_pos, int n_tok, int H, int G, int Gv,
+                                   int dk, int dv, int block_size, int64_t max_blocks, int dtype, void* stream) {
   if (Gv <= 0) return fail(B200_EINVAL, "b200_qknorm_rotary_append: bad sizes");
   if (n_tok < 0 || H <= 0 || G <= 0 || dk <= 0 || dv <= 0 || block_size <= 0 || max_blocks <= 0)
     return fail(B200_EINVAL, "b200_qknorm_rotary_append: bad sizes");
@@ -610,7 +620,7 @@ int b200_qknorm_rotary_append_ext(void* q, int64_t q_stride, const void* k, int6
     if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     kern<<<n_tok, kQkWarps * 32, smem, static_cast<cudaStream_t>(stream)>>>(
         static_cast<T*>(q), q_stride, static_cast<const T*>(k), k_stride, static_cast<const T*>(v), v_stride,
-        static_cast<const T*>(q_norm), static_cast<const T*>(k_norm), eps, freqs, rot_dims, interleaved,
+        static_cast<const T*>(q_norm), static_cast<const T*>(k_norm), unit_norm, eps, freqs, rot_dims, interleaved,
         static_cast<T*>(k_pool), static_cast<T*>(v_pool), slot_mapping, tok_pos, H, G, Gv, dk, dv, block_size);
     return check_launch("b200_qknorm_rotary_append");
   });

@@ -387,6 +387,15 @@ def norm_append(x: torch.Tensor, weight: torch.Tensor, eps: float, pool: torch.T
     _lib.check_mixers(rc, "b200_norm_append")
 
 
+def _gate_kind(gate: Optional[torch.Tensor], n: int, H: int, dv: int, dtype: torch.dtype) -> int:
+    """0: no gate, or one per head (``[n, H]``); 1: one per output channel (``[n, H*dv]``)."""
+    if gate is None:
+        return 0
+    if gate.dtype != dtype or tuple(gate.shape) not in ((n, H), (n, H * dv)):
+        raise ValueError("gate must be [n, H] or [n, H*dv] in the activations' dtype")
+    return int(gate.shape[1] != H)
+
+
 def _value_layout(k_pool: torch.Tensor, v_pool: torch.Tensor, value_width: Optional[int], value_div: int):
     """``(value size, elements between value rows)`` of an attention call, after checking the pools against each other."""
     if v_pool.dim() != 4 or v_pool.shape[0] != k_pool.shape[0] or v_pool.shape[2] != k_pool.shape[2]:
@@ -411,7 +420,8 @@ def mixed_paged_attention(out: torch.Tensor, q: torch.Tensor, k_pool: torch.Tens
     VIEWS with a contiguous last dimension (any token / head strides); ``talk`` fp32 ``[H, H]`` mixes the heads'
     scores before the softmax, ``sink`` fp32 ``[H]`` adds exp(sink) to the denominator, ``window`` > 0 limits a
     position to its last ``window`` tokens plus the sequence's first ``keep_first``, ``unrotate_base`` turns the
-    output back by the position over the value width, ``gate`` ``[n, H]`` is a sigmoid gate per head, ``softcap`` > 0
+    output back by the position over the value width, ``gate`` holds the logits of a sigmoid gate per head (``[n, H]``) or
+    per output channel (``[n, H*dv]``, not with ``unrotate_base``), ``softcap`` > 0
     bounds the scores by ``softcap * tanh(score / softcap)`` before the mask, ``chunk`` > 0 lets a position see only
     the keys of its own block of ``chunk`` positions, ``value_width`` says that the values are the first that many
     columns of the (wider) rows of ``v_pool``, ``value_div`` that ``v_pool`` holds one value head per that many key
@@ -432,10 +442,9 @@ def mixed_paged_attention(out: torch.Tensor, q: torch.Tensor, k_pool: torch.Tens
     for t, shape in ((talk, (H, H)), (sink, (H,))):
         if t is not None and (t.dtype != torch.float32 or tuple(t.shape) != shape or not t.is_contiguous()):
             raise ValueError("talk is contiguous fp32 [H, H], sink fp32 [H]")
-    if gate is not None and (tuple(gate.shape) != (n, H) or gate.dtype != q.dtype):
-        raise ValueError("gate must be [n, H] in the activations' dtype")
-    rc = _lib_().b200_mixed_paged_attn_ext(out.data_ptr(), out.stride(0), out.stride(1), q.data_ptr(), q.stride(0),
-                                           q.stride(1), _ptr(gate), _rows2(gate) if gate is not None else 0,
+    per_channel = _gate_kind(gate, n, H, dv, q.dtype)
+    rc = _lib_().b200_mixed_paged_attn_ext2(out.data_ptr(), out.stride(0), out.stride(1), q.data_ptr(), q.stride(0),
+                                           q.stride(1), _ptr(gate), _rows2(gate) if gate is not None else 0, per_channel,
                                            k_pool.data_ptr(), v_pool.data_ptr(), block_tables.data_ptr(),
                                            block_tables.stride(0), tok_row.data_ptr(), tok_pos.data_ptr(), n, _ptr(talk),
                                            _ptr(sink), float(scale), float(softcap), int(window), int(keep_first),
@@ -449,6 +458,11 @@ def mixed_prompt_attention_supported(H: int, G: int, dk: int, dv: int, has_talk:
                                      dtype: torch.dtype) -> bool:
     return bool(_lib_().b200_mixed_prompt_attn_supported(int(H), int(G), int(dk), int(dv), int(has_talk), int(same_pool),
                                                          int(unrotate), DTYPE_ID[dtype]))
+
+
+def heads_as_rows_supported(H: int, G: int, dk: int, dv: int, dtype: torch.dtype) -> bool:
+    """Whether ``mixed_prompt_attention(heads_as_rows=True)`` takes this head layout."""
+    return bool(_lib_().b200_mixed_prompt_attn_rows_supported(int(H), int(G), int(dk), int(dv), DTYPE_ID[dtype]))
 
 
 PROMPT_TILE_TOKENS = 16     # tokens of one sequence a CTA of ``mixed_prompt_attention`` serves
@@ -467,8 +481,9 @@ def mixed_prompt_attention(out: torch.Tensor, q: torch.Tensor, k_pool: torch.Ten
     tokens of one sequence each, together covering every row of ``q``; ``value_rot``: the table ``rotary_kv_append``
     returned for this step's tokens; ``max_context``: the longest context of the step (a hint: steps of few tokens over
     long contexts divide the keys over several CTAs and merge); ``chunk``, ``value_width`` and ``value_div`` as in
-    ``mixed_paged_attention``.  ``heads_as_rows`` (steps of single tokens over one kv head, no talk / gate / value_rot):
-    the 16 rows of a tensor-core tile are 16 query heads of one token instead of 16 tokens of one head."""
+    ``mixed_paged_attention``, as are the kinds of ``gate``.  ``heads_as_rows`` (steps of single tokens, no talk / value_rot /
+    value_div; see ``heads_as_rows_supported``): the 16 rows of a tensor-core tile are up to 16 query heads of one token that
+    share a kv head instead of 16 tokens of one head."""
     _need_cuda(out, q, k_pool, v_pool, block_tables, tiles, tok_pos)
     nb, G, bs, dk = k_pool.shape
     dv, v_row = _value_layout(k_pool, v_pool, value_width, value_div)
@@ -486,23 +501,23 @@ def mixed_prompt_attention(out: torch.Tensor, q: torch.Tensor, k_pool: torch.Ten
     if value_rot is not None and (tuple(value_rot.shape) != (n, dv // 2, 2) or value_rot.dtype != torch.float32
                                   or not value_rot.is_contiguous()):
         raise ValueError("value_rot must be contiguous fp32 [n, dv // 2, 2]")
-    if gate is not None and (tuple(gate.shape) != (n, H) or gate.dtype != q.dtype):
-        raise ValueError("gate must be [n, H] in the activations' dtype")
-    if heads_as_rows and (G != 1 or talk is not None or gate is not None or value_rot is not None):
-        raise ValueError("heads_as_rows needs one kv head and no talk, gate or value_rot")
+    per_channel = _gate_kind(gate, n, H, dv, q.dtype)
+    if heads_as_rows and (H % G or talk is not None or value_rot is not None or value_div != 1):
+        raise ValueError("heads_as_rows goes with no talk, value_rot or value_div")
+    rows_heads = G * ((H // G + 15) // 16) if heads_as_rows else H
     lib = _lib_()
     seen = min(max_context, window + keep_first + PROMPT_TILE_TOKENS) if window > 0 else max_context
     if chunk > 0:
         seen = min(seen, chunk + PROMPT_TILE_TOKENS)
-    splits = lib.b200_mixed_prompt_attn_splits(tiles.shape[0], (seen + 31) // 32, (H + 15) // 16 if heads_as_rows else H, G,
+    splits = lib.b200_mixed_prompt_attn_splits(tiles.shape[0], (seen + 31) // 32, rows_heads, G,
                                                dk, dv, int(talk is not None),
                                                int(k_pool.data_ptr() == v_pool.data_ptr()), int(value_rot is not None),
                                                DTYPE_ID[q.dtype]) if max_context > 0 else 1
     ws = None
     if splits > 1:
         ws = torch.empty(lib.b200_mixed_prompt_attn_workspace(splits, n, H, dv) // 4, dtype=torch.float32, device=q.device)
-    rc = lib.b200_mixed_prompt_attn_ext(out.data_ptr(), out.stride(0), out.stride(1), q.data_ptr(), q.stride(0),
-                                        q.stride(1), _ptr(gate), _rows2(gate) if gate is not None else 0, k_pool.data_ptr(),
+    rc = lib.b200_mixed_prompt_attn_ext2(out.data_ptr(), out.stride(0), out.stride(1), q.data_ptr(), q.stride(0),
+                                        q.stride(1), _ptr(gate), _rows2(gate) if gate is not None else 0, per_channel, k_pool.data_ptr(),
                                         v_pool.data_ptr(), block_tables.data_ptr(), block_tables.stride(0),
                                         tiles.data_ptr(), tiles.shape[0], tok_pos.data_ptr(), n, _ptr(talk), _ptr(sink),
                                         float(scale), float(softcap), int(window), int(keep_first), int(chunk),
@@ -538,16 +553,21 @@ def causal_conv_silu(x: torch.Tensor, weight: torch.Tensor, tail: torch.Tensor, 
 @_timed
 def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta_logit: torch.Tensor, a_logit: torch.Tensor,
                dt_bias: torch.Tensor, a_log: torch.Tensor, state: torch.Tensor, seqs: torch.Tensor, G: int,
-               unit_eps: float, q_scale: float) -> torch.Tensor:
-    """Gated delta rule with a decay per key channel over each sequence's tokens; ``state`` fp32 ``[slots, H, dk, dv]``
+               unit_eps: float, q_scale: float, max_count: int = 0) -> torch.Tensor:
+    """Gated delta rule with a decay per key channel (``a_logit [n, H*dk]``, ``dt_bias [H*dk]``) or per head (``[n, H]``,
+    ``[H]``) over each sequence's tokens; ``state`` fp32 ``[slots, H, dk, dv]``
     is read (unless the sequence is fresh) and written back.  ``q / k [n, G*dk]`` and ``v [n, H*dv]`` are column
-    slices of ONE tensor (same row stride), ``beta_logit [n, H]``, ``a_logit [n, H*dk]``.  Returns fp32 ``[n, H, dv]``."""
+    slices of ONE tensor (same row stride), ``beta_logit [n, H]``.  Returns fp32 ``[n, H, dv]``.  ``max_count``: the
+    largest token count in ``seqs`` (0: unknown); with one decay per head it picks the kernel: steps of single tokens, bf16
+    steps with a portion of ``CHUNK_SCAN_FROM`` tokens or more in chunks on the tensor cores, others token by token."""
     _need_cuda(q, k, v, beta_logit, a_logit, dt_bias, a_log, state, seqs)
     n = q.shape[0]
     _, H, dk, dv = state.shape
     if q.shape[1] != G * dk or k.shape != q.shape or v.shape != (n, H * dv) or beta_logit.shape != (n, H) \
-            or a_logit.shape != (n, H * dk) or dt_bias.numel() != H * dk or a_log.numel() != H:
+            or a_log.numel() != H or (tuple(a_logit.shape), dt_bias.numel()) not in (((n, H * dk), H * dk), ((n, H), H)):
         raise ValueError("inputs do not match the state's shape")
+    if any(t.dtype != q.dtype for t in (k, v, beta_logit, a_logit, dt_bias, a_log)):
+        raise TypeError("inputs and constants share one dtype")
     stride = _rows2(q)
     if n > 1 and (k.stride(0) != stride or v.stride(0) != stride):
         raise ValueError("q, k and v must share a row stride")
@@ -556,11 +576,22 @@ def delta_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta_logit: to
     if seqs.dtype != torch.int32 or seqs.dim() != 2 or seqs.shape[1] != 4 or not seqs.is_contiguous():
         raise ValueError("seqs must be contiguous int32 [n_seqs, 4]")
     o = torch.empty((n, H, dv), dtype=torch.float32, device=q.device)
-    rc = _lib_().b200_delta_scan(o.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(), stride, beta_logit.data_ptr(),
-                                 _rows2(beta_logit), a_logit.data_ptr(), _rows2(a_logit), dt_bias.data_ptr(),
-                                 a_log.data_ptr(), state.data_ptr(), seqs.data_ptr(), seqs.shape[0], H, G, dk, dv,
-                                 float(unit_eps), float(q_scale), DTYPE_ID[q.dtype], _stream())
-    _lib.check_mixers(rc, "b200_delta_scan")
+    lib, dt, n_seqs = _lib_(), DTYPE_ID[q.dtype], seqs.shape[0]
+    head = (o.data_ptr(), q.data_ptr(), k.data_ptr(), v.data_ptr(), stride, beta_logit.data_ptr(), _rows2(beta_logit),
+            a_logit.data_ptr(), _rows2(a_logit), dt_bias.data_ptr(), a_log.data_ptr())
+    tail = (H, G, dk, dv, float(unit_eps), float(q_scale))
+    one_decay = a_logit.shape[1] == H
+    if one_decay and max_count == 1 and n_seqs == n:
+        rc = lib.b200_delta_step(*head, state.data_ptr(), seqs.data_ptr(), n_seqs, *tail, dt, _stream())
+        _lib.check_mixers(rc, "b200_delta_step")
+    elif one_decay and max_count >= CHUNK_SCAN_FROM and lib.b200_delta_chunk_scan_supported(dk, dv, dt):
+        ws = torch.empty(lib.b200_delta_chunk_workspace(n, n_seqs, H), dtype=torch.uint8, device=q.device)
+        rc = lib.b200_delta_chunk_scan(*head, state.data_ptr(), seqs.data_ptr(), n_seqs, int(max_count), *tail, ws.data_ptr(), dt,
+                                       _stream())
+        _lib.check_mixers(rc, "b200_delta_chunk_scan")
+    else:
+        rc = lib.b200_delta_scan_ext(*head, int(not one_decay), state.data_ptr(), seqs.data_ptr(), n_seqs, *tail, dt, _stream())
+        _lib.check_mixers(rc, "b200_delta_scan")
     return o
 
 
@@ -592,8 +623,9 @@ def _check_seqs(seqs: torch.Tensor) -> None:
 def qknorm_rotary_append(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_norm: Optional[torch.Tensor],
                          k_norm: Optional[torch.Tensor], eps: float, freqs: Optional[torch.Tensor], k_pool: torch.Tensor,
                          v_pool: torch.Tensor, slot_mapping: torch.Tensor, tok_pos: torch.Tensor, H: int,
-                         interleaved: bool = True) -> None:
-    """Per-head RMS norm of q (in place) and k (weights ``[dk]``, None: no norm), rotary positions over the first
+                         interleaved: bool = True, unit_norm: bool = False) -> None:
+    """Per-head RMS norm of q (in place) and k (weights ``[dk]``; None: no norm, or with ``unit_norm`` a norm without a
+    weight, which a rotation leaves as it is), rotary positions over the first
     ``2 * len(freqs)`` dimensions of every head with angle ``pos * freqs[i]`` (``freqs`` float64 on the device), k and v
     stored in the pools at ``slot_mapping``.  ``v_pool`` may hold fewer heads than ``k_pool`` (several score maps over the
     same values)."""
@@ -614,8 +646,8 @@ def qknorm_rotary_append(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_no
         if freqs.dtype != torch.float64 or not freqs.is_contiguous() or not freqs.is_cuda:
             raise ValueError("freqs is a contiguous float64 tensor on the device")
         rot_dims = 2 * freqs.numel()
-    rc = _lib_().b200_qknorm_rotary_append_ext(q.data_ptr(), _rows2(q), k.data_ptr(), _rows2(k), v.data_ptr(), _rows2(v),
-                                               _ptr(q_norm), _ptr(k_norm), float(eps), _ptr(freqs), rot_dims,
+    rc = _lib_().b200_qknorm_rotary_append_ext2(q.data_ptr(), _rows2(q), k.data_ptr(), _rows2(k), v.data_ptr(), _rows2(v),
+                                               _ptr(q_norm), _ptr(k_norm), int(unit_norm), float(eps), _ptr(freqs), rot_dims,
                                                int(interleaved), k_pool.data_ptr(), v_pool.data_ptr(),
                                                slot_mapping.data_ptr(), tok_pos.data_ptr(), n, H, G, Gv, dk, dv, bs, nb,
                                                DTYPE_ID[k_pool.dtype], _stream())
@@ -1189,3 +1221,74 @@ def gated_part_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, eps:
                                       inner, int(parts), DTYPE_ID[weight.dtype], _stream())
     _lib.check_mixers(rc, "b200_gated_part_norm")
     return out
+
+
+# ---- per-channel selective state spaces, sublayers normed on both sides (csrc/b200_selective_ops.cu) --------------------
+@_timed
+def selective_scan(x: torch.Tensor, dt: torch.Tensor, B: torch.Tensor, C: torch.Tensor, z: torch.Tensor, dt_bias: torch.Tensor,
+                   a_log: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, seqs: torch.Tensor, gain: float = 1.0,
+                   out: Optional[torch.Tensor] = None, max_count: int = 0) -> torch.Tensor:
+    """Per channel ``c`` and state ``n``, with ``dt = softplus(dt + dt_bias)``: ``S <- e^(-e^a_log dt) S + dt x B``, ``y = S.C +
+    skip x``; returns ``gain * y * silu(z)`` ``[n, inner]`` in the activations' dtype (``out`` may be a column slice of a wider
+    buffer).  ``x / dt / z [n, inner]`` and ``B / C [n, N]`` (one row stride) may be column slices; ``dt_bias``, ``skip`` fp32
+    ``[inner]``, ``a_log`` fp32 ``[inner, N]``, ``state`` fp32 ``[slots, inner, N]``.  ``max_count``: the largest token count in
+    ``seqs``; steps of single tokens take a launch of their own."""
+    _need_cuda(x, dt, B, C, z, state, seqs)
+    _check_seqs(seqs)
+    n, inner = x.shape
+    N = B.shape[1]
+    if dt.shape != x.shape or z.shape != x.shape or B.shape != (n, N) or C.shape != B.shape:
+        raise ValueError("x, dt, z are [n, inner], B and C [n, N]")
+    if n > 1 and B.stride(0) != C.stride(0):
+        raise ValueError("B and C must share a row stride")
+    if any(t.dtype != x.dtype for t in (dt, B, C, z)):
+        raise TypeError("activations share one dtype")
+    for t, shape in ((dt_bias, (inner,)), (skip, (inner,)), (a_log, (inner, N)), (state, (state.shape[0], inner, N))):
+        if t.dtype != torch.float32 or tuple(t.shape) != shape or not t.is_contiguous():
+            raise ValueError("constants and state are contiguous fp32")
+    if out is None:
+        out = torch.empty((n, inner), dtype=x.dtype, device=x.device)
+    elif out.shape != x.shape or out.dtype != x.dtype:
+        raise ValueError("out must be [n, inner] in the activations' dtype")
+    step = max_count == 1 and seqs.shape[0] == n
+    fn = _lib_().b200_selective_step if step else _lib_().b200_selective_scan
+    rc = fn(out.data_ptr(), _rows2(out), x.data_ptr(), _rows2(x), dt.data_ptr(), _rows2(dt), dt_bias.data_ptr(), a_log.data_ptr(),
+            B.data_ptr(), C.data_ptr(), _rows2(B), skip.data_ptr(), z.data_ptr(), _rows2(z), float(gain), state.data_ptr(),
+            seqs.data_ptr(), seqs.shape[0], inner, N, DTYPE_ID[x.dtype], _stream())
+    _lib.check_mixers(rc, "b200_selective_step" if step else "b200_selective_scan")
+    return out
+
+
+@_timed
+def sandwich_residual(x: torch.Tensor, y: torch.Tensor, w_norm: torch.Tensor, layer_scale: Optional[torch.Tensor], eps: float,
+                      w_next: Optional[torch.Tensor] = None, eps_next: float = 0.0, sign: float = 1.0) -> Optional[torch.Tensor]:
+    """In place ``x += sign * layer_scale * w_norm * y * rsqrt(mean(y^2) + eps)`` on the fp32 residual (``y`` fp32 or of the
+    weights' dtype); with ``w_next`` returns ``w_next * x * rsqrt(mean(x^2) + eps_next)`` of the new residual in that dtype."""
+    _need_cuda(x, y, w_norm)
+    T = w_norm.dtype
+    if x.dtype != torch.float32 or not x.is_contiguous() or x.dim() != 2 or y.shape != x.shape:
+        raise ValueError("x must be contiguous fp32 [rows, width] and y of the same shape")
+    if y.dtype not in (T, torch.float32):
+        raise TypeError("y is fp32 or of the weights' dtype")
+    for w in (w_norm, layer_scale, w_next):
+        if w is not None and (w.dtype != T or w.numel() != x.shape[1] or not w.is_contiguous()):
+            raise ValueError("weights are contiguous [width] in one dtype")
+    out = torch.empty(x.shape, dtype=T, device=x.device) if w_next is not None else None
+    rc = _lib_().b200_sandwich_residual(x.data_ptr(), y.data_ptr(), _rows2(y), int(y.dtype == torch.float32 and T != torch.float32),
+                                        float(sign), w_norm.data_ptr(), _ptr(layer_scale), float(eps), _ptr(w_next),
+                                        float(eps_next), _ptr(out), x.shape[0], x.shape[1], DTYPE_ID[T], _stream())
+    _lib.check_mixers(rc, "b200_sandwich_residual")
+    return out
+
+
+@_timed
+def gelu_glu(gu: torch.Tensor) -> torch.Tensor:
+    """``gelu_tanh(g) * u`` of contiguous rows ``g | u``."""
+    _need_cuda(gu)
+    if not gu.is_contiguous() or gu.dim() != 2 or gu.shape[1] % 2:
+        raise ValueError("gu must be contiguous [rows, 2*ff]")
+    ff = gu.shape[1] // 2
+    y = torch.empty((gu.shape[0], ff), dtype=gu.dtype, device=gu.device)
+    rc = _lib_().b200_gelu_glu(y.data_ptr(), gu.data_ptr(), gu.shape[0], ff, DTYPE_ID[gu.dtype], _stream())
+    _lib.check_mixers(rc, "b200_gelu_glu")
+    return y

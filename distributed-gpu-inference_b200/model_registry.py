@@ -69,7 +69,7 @@ def _register_builtin() -> None:
     if _builtin_done:
         return
     _builtin_done = True
-    from . import fibirax_layer, petipel_layer, sanesun_layer, vatazen_layer, zuderax_layer
+    from . import fibirax_layer, petipel_layer, rufedra_layer, sanesun_layer, vatazen_layer, zuderax_layer
     from .testing import LlamaShapeConfig, build_product_shards
 
     def llama_config(raw: Dict[str, Any]):
@@ -83,3 +83,4 @@ def _register_builtin() -> None:
     register(Architecture("Fibirax", fibirax_layer.FibiraxConfig.from_dict, fibirax_layer.build_shards, "ragged"))
     register(Architecture("Vatazen", vatazen_layer.VatazenConfig.from_dict, vatazen_layer.build_shards, "ragged"))
     register(Architecture("Zuderax", zuderax_layer.ZuderaxConfig.from_dict, zuderax_layer.build_shards, "ragged"))
+    register(Architecture("Rufedra", rufedra_layer.RufedraConfig.from_dict, rufedra_layer.build_shards, "ragged"))

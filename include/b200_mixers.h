@@ -443,6 +443,90 @@ int b200_normalized_head_out(void* out, int64_t out_stride, const float* o, cons
 int b200_gated_part_norm(void* out, const float* y, const void* z, int64_t z_stride, const void* w, float eps, int64_t n_tok,
                          int inner, int parts, int dtype, void* stream);
 
+/* b200_mixed_paged_attn_ext with gate_per_channel: != 0: gate rows hold H * dv logits, out(i, h, c) *= sigmoid(gate[i][h * dv + c])
+ * (not with unrotate). */
+int b200_mixed_paged_attn_ext2(void* out, int64_t out_tok_stride, int64_t out_head_stride, const void* q,
+                               int64_t q_tok_stride, int64_t q_head_stride, const void* gate, int64_t gate_stride,
+                               int gate_per_channel, const void* k_pool, const void* v_pool, const int32_t* block_tables,
+                               int table_stride, const int32_t* tok_row, const int32_t* tok_pos, int n_tok,
+                               const float* talk, const float* sink, float scale, float softcap, int window, int keep_first,
+                               int chunk, int unrotate, int interleaved, float rot_base, int H, int G, int dk, int dv,
+                               int v_row, int v_div, int out_f32, int block_size, int dtype, void* stream);
+
+/* b200_mixed_prompt_attn_ext with gate_per_channel as above (not with value_rot), and heads_as_rows for any number of kv heads:
+ * the 16 rows of a tensor-core tile are up to 16 of the H / G query heads that share a kv head, with gates of either kind.  For
+ * b200_mixed_prompt_attn_splits such a step counts G * ceil(H / G / 16) heads. */
+int b200_mixed_prompt_attn_ext2(void* out, int64_t out_tok_stride, int64_t out_head_stride, const void* q,
+                                int64_t q_tok_stride, int64_t q_head_stride, const void* gate, int64_t gate_stride,
+                                int gate_per_channel, const void* k_pool, const void* v_pool, const int32_t* block_tables,
+                                int table_stride, const int32_t* tiles, int n_tiles, const int32_t* tok_pos, int n_tok,
+                                const float* talk, const float* sink, float scale, float softcap, int window,
+                                int keep_first, int chunk, const float* value_rot, int interleaved, int H, int G, int dk,
+                                int dv, int v_row, int v_div, int heads_as_rows, int out_f32, int block_size, int n_splits,
+                                float* workspace, int dtype, void* stream);
+
+/* Whether b200_mixed_prompt_attn_ext2 takes this layout with heads_as_rows (separate key and value pools). */
+int b200_mixed_prompt_attn_rows_supported(int H, int G, int dk, int dv, int dtype);
+
+/* b200_qknorm_rotary_append_ext with unit_norm: != 0: q and k rows are divided by their RMS even where q_norm / k_norm is NULL
+ * (a norm without a weight: before or after the rotation is the same). */
+int b200_qknorm_rotary_append_ext2(void* q, int64_t q_stride, const void* k, int64_t k_stride, const void* v,
+                                   int64_t v_stride, const void* q_norm, const void* k_norm, int unit_norm, float eps,
+                                   const double* freqs, int rot_dims, int interleaved, void* k_pool, void* v_pool,
+                                   const int64_t* slot_mapping, const int32_t* tok_pos, int n_tok, int H, int G, int Gv,
+                                   int dk, int dv, int block_size, int64_t max_blocks, int dtype, void* stream);
+
+/* b200_delta_scan with per_channel as an argument: 1: a_logit T [n, H*dk] and dt_bias T [H*dk]; 0: ONE decay per token and head,
+ * a_logit T [n, H] and dt_bias T [H]. */
+int b200_delta_scan_ext(float* o_raw, const void* q, const void* k, const void* v, int64_t in_stride, const void* beta_logit,
+                        int64_t beta_stride, const void* a_logit, int64_t a_stride, const void* dt_bias, const void* a_log,
+                        int per_channel, float* state, const int32_t* seqs, int n_seqs, int H, int G, int dk, int dv,
+                        float unit_eps, float q_scale, int dtype, void* stream);
+
+/* ---- the delta rule with one decay per head in chunks, and per-channel selective state spaces ---------------------- */
+
+/* b200_delta_scan_ext with per_channel = 0 in chunks of 64 tokens on the tensor cores (bf16, dk <= 256): q, k and v enter the
+ * products as they are, fp32 operands as the sum of two bf16 numbers, accumulation and state are fp32.  The rows of seqs are in
+ * the order of their tokens; max_count: the largest token count among them; workspace: b200_delta_chunk_workspace bytes, 16-byte
+ * aligned (n_tok: the step's tokens). */
+int b200_delta_chunk_scan_supported(int dk, int dv, int dtype);
+size_t b200_delta_chunk_workspace(int n_tok, int n_seqs, int H);
+int b200_delta_chunk_scan(float* o_raw, const void* q, const void* k, const void* v, int64_t in_stride, const void* beta_logit,
+                          int64_t beta_stride, const void* a_logit, int64_t a_stride, const void* dt_bias, const void* a_log,
+                          float* state, const int32_t* seqs, int n_seqs, int max_count, int H, int G, int dk, int dv,
+                          float unit_eps, float q_scale, void* workspace, int dtype, void* stream);
+
+/* The same for steps whose sequences bring ONE token each (any dtype): the state is read and written once. */
+int b200_delta_step(float* o_raw, const void* q, const void* k, const void* v, int64_t in_stride, const void* beta_logit,
+                    int64_t beta_stride, const void* a_logit, int64_t a_stride, const void* dt_bias, const void* a_log,
+                    float* state, const int32_t* seqs, int n_seqs, int H, int G, int dk, int dv, float unit_eps, float q_scale,
+                    int dtype, void* stream);
+
+/* Selective state space per (sequence, channel c) over the sequence's tokens of this step, in order (SeqSpan rows):
+ *   dt = softplus(dt_logit + dt_bias);  S[c, n] <- exp(-exp(a_log[c, n]) dt_c) S[c, n] + dt_c x_c B_n;
+ *   out_c = gain * (sum_n S[c, n] C_n + skip_c x_c) * silu(z_c)
+ * x, dt, z: T rows of `inner`; b, c: T rows of n_state with one row stride; out T rows; dt_bias, skip fp32 [inner]; a_log fp32
+ * [inner, n_state]; state fp32 [slots, inner, n_state], read unless the sequence is fresh and written back.  n_state <= 256. */
+int b200_selective_scan(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* dt, int64_t dt_stride,
+                        const float* dt_bias, const float* a_log, const void* b, const void* c, int64_t bc_stride,
+                        const float* skip, const void* z, int64_t z_stride, float gain, float* state, const int32_t* seqs,
+                        int n_seqs, int inner, int n_state, int dtype, void* stream);
+
+/* The same for steps whose sequences bring ONE token each (any n_state). */
+int b200_selective_step(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* dt, int64_t dt_stride,
+                        const float* dt_bias, const float* a_log, const void* b, const void* c, int64_t bc_stride,
+                        const float* skip, const void* z, int64_t z_stride, float gain, float* state, const int32_t* seqs,
+                        int n_seqs, int inner, int n_state, int dtype, void* stream);
+
+/* x[r] += sign * layer_scale * w_norm * y[r] * rsqrt(mean(y[r]^2) + eps)  in place on the fp32 residual (layer_scale T [width] may
+ * be NULL; y T, or fp32 with y_is_f32); out[r] = w_next * x[r] * rsqrt(mean(x[r]^2) + eps_next) in T (out may be NULL). */
+int b200_sandwich_residual(float* x, const void* y, int64_t y_stride, int y_is_f32, float sign, const void* w_norm,
+                           const void* layer_scale, float eps, const void* w_next, float eps_next, void* out, int rows,
+                           int width, int dtype, void* stream);
+
+/* y = gelu_tanh(g) * u; gu rows = g | u, contiguous [rows, 2 * ff]. */
+int b200_gelu_glu(void* y, const void* gu, int64_t rows, int ff, int dtype, void* stream);
+
 #ifdef __cplusplus
 }
 #endif
