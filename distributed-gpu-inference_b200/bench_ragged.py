@@ -23,6 +23,11 @@ attention on the same tensor-core kernel, softmax routing over the same dispatch
 routed experts with a shared expert in every layer) beside the two models that have its like kernels, at equal width, depth,
 head layout and expert sizes: Fibirax (a decayed outer-product state per head in every layer, grouped routing, a shared
 expert) and Vatazen (the same latent attention).
+
+``bench.py --compare rufedra``: the same two steps for the Rufedra model class (gated delta rules in turn with layers that run a
+windowed attention beside a selective state space, dense feed-forwards) beside the models that have its like kernels, at equal
+width, depth and head layout: Sanesun (a delta rule behind short convolutions, windowed attention, dense feed-forwards of the same
+size), Fibirax (windowed attention beside a recurrence in every layer, post-norms) and Zuderax (a state space per head).
 """
 from __future__ import annotations
 
@@ -751,6 +756,104 @@ def _zuderax_kernel_table(s, ev_prompt, ev_decode, B, Pn, Bd, ctx, hbm, tf) -> D
             "silu_glu[shared]": (n_tok * eff * 6, 0),
             "router_logits": (n_tok * W * 2, 0),
             "gather_rows": (n_tok * top * W * 4, 0),
+        }
+        for name, ts in by.items():
+            t = statistics.mean(ts)
+            entry = {"us": round(t * 1e6, 1), "calls": len(ts)}
+            if name in floors:
+                nbytes, flops = floors[name]
+                floor = max(nbytes / hbm, flops / tf)
+                entry["of_floor"] = round(floor / t, 3)
+                entry["bound"] = "math" if flops / tf > nbytes / hbm else "memory"
+            out.setdefault(phase, {})[name] = entry
+    return out
+
+
+# ---- Rufedra beside Sanesun, Fibirax and Zuderax ---------------------------------------------------------------------
+RUFEDRA_WINDOW = 512
+RUFEDRA_STATE, RUFEDRA_CONV = 16, 4
+
+
+def rufedra_config(s: Dict[str, int]) -> Dict[str, Any]:
+    """Delta layers take the size's recurrent heads (two value heads per q / k head); the state space is twice as wide as the
+    model, with 16 states per channel and a step-size rank of a sixteenth of the width."""
+    rec = {"type": "delta", "mixer": {"heads": s["rheads"], "kv_heads": s["rheads"] // 2, "dim": s["rdk"], "vdim": s["rdv"],
+                                      "conv": RUFEDRA_CONV}}
+    par = {"type": "parallel", "mixer": {
+        "left": {"heads": s["heads"], "kv_heads": s["kv"], "dim": s["dk"], "vdim": s["dk"], "scale": 1.0 / math.sqrt(s["dk"]),
+                 "mask": {"size": RUFEDRA_WINDOW}, "rot": {"base": 10000.0, "dims": s["dk"] // 2}},
+        "right": {"inner": 2 * s["width"], "state": RUFEDRA_STATE, "dt_rank": s["width"] // 16, "conv": RUFEDRA_CONV},
+        "left_scale": 0.8, "right_scale": 0.5}}
+    return {"architecture": "Rufedra", "width": s["width"], "vocab": VOCAB, "embedding": {"scale": 1.0}, "norm": {"eps": 1e-6},
+            "logit_scale": 1.0, "layers": [dict(m, mlp={"kind": "dense", "ff": s["ff"]}) for m in (rec, par, rec, par)]}
+
+
+def run_rufedra(args, measured_peaks, ClockSampler) -> None:
+    from . import fibirax_layer as Fx
+    from . import rufedra_layer as Q
+    from . import sanesun_layer as Sn
+    from . import zuderax_layer as Z
+
+    peaks, how = measured_peaks()
+    hbm, tf = peaks["hbm_gbs"] * 1e9, peaks["bf16_tflops"] * 1e12
+    steps, warmup = max(3, args.steps), max(3, args.warmup)
+    B, Pn, ctx, Bd = 8, 2048, 2048, 64
+    g = torch.Generator().manual_seed(0)
+    sampler = ClockSampler(0)
+    sampler.start()
+    report: Dict[str, Any] = {}
+    for name, s in SIZES.items():
+        if args.compare_sizes and name not in args.compare_sizes.split(","):
+            continue
+        row: Dict[str, Any] = {}
+        prompts = torch.randint(0, VOCAB, (Bd, ctx), generator=g).tolist()
+        for label, mod, cfg, table in (
+                ("rufedra", Q, Q.RufedraConfig(rufedra_config(s)), _rufedra_kernel_table),
+                ("sanesun", Sn, Sn.SanesunConfig(sanesun_config(s)), _sanesun_kernel_table),
+                ("fibirax", Fx, Fx.FibiraxConfig(fibirax_config(s)), _fibirax_kernel_table),
+                ("zuderax", Z, Z.ZuderaxConfig(zuderax_config(s)), _zuderax_kernel_table)):
+            prefill, decode, kernels = _measure_ragged(mod, cfg, table, s, B, Pn, Bd, ctx, steps, warmup, prompts, hbm, tf)
+            row[label + "_prefill_tok_s"], row[label + "_decode_tok_s"], row[label + "_kernels"] = prefill, decode, kernels
+            torch.cuda.empty_cache()
+        row["inputs_exceed_l2"] = bool(Bd * s["rheads"] * s["rdk"] * s["rdv"] * 4 * LAYERS > 126e6)
+        report[name] = row
+    clocks = sampler.stop()
+    print(json.dumps({"bench": "rufedra_vs_sanesun_fibirax_and_zuderax", "unit": "tokens/s", "dtype": "bf16", "data": "synthetic",
+                      "layers": LAYERS, "prompt_step": f"{B} x {Pn} tokens", "decode_step": f"{Bd} sequences at {ctx}",
+                      "peaks": how, "sizes": report, "clocks": clocks}), flush=True)
+
+
+def _rufedra_kernel_table(s, ev_prompt, ev_decode, B, Pn, Bd, ctx, hbm, tf) -> Dict[str, Any]:
+    """Like ``_kernel_table`` for the Rufedra kernels.  Calls of the convolution are listed per layer type (delta layers come
+    first and in turn with parallel ones)."""
+    out: Dict[str, Any] = {}
+    W, H, G, dk = s["width"], s["heads"], s["kv"], s["dk"]
+    RH, RG, rdk, rdv = s["rheads"], s["rheads"] // 2, s["rdk"], s["rdv"]
+    inner, N = 2 * W, RUFEDRA_STATE
+    C = 2 * RG * rdk + RH * rdv
+    for phase, events, n_tok, past in (("prompt", ev_prompt, B * Pn, 0), ("decode", ev_decode, Bd, ctx)):
+        by: Dict[str, List[float]] = {}
+        convs = 0
+        for name, a, b in events:
+            if name == "causal_conv_silu":
+                name += "[delta]" if convs % 2 == 0 else "[parallel]"
+                convs += 1
+            by.setdefault(name, []).append(a.elapsed_time(b) * 1e-3)
+        per_seq = n_tok // (B if phase == "prompt" else Bd)
+        n_seq = n_tok // per_seq
+        pairs = sum(min(past + t + 1, RUFEDRA_WINDOW) for t in range(per_seq))
+        keys = min(past + per_seq, RUFEDRA_WINDOW + per_seq)
+        floors = {
+            "rms_norm": (n_tok * W * 6, 0),
+            "sandwich_residual": (n_tok * W * (4 + 4 + 2 + 2), 0),
+            "qknorm_rotary_append": (n_tok * (H * dk * 2 + G * (dk + dk) * 2) * 2, 0),
+            "mixed_prompt_attention": (n_seq * keys * G * 2 * dk * 2 + n_tok * H * 3 * dk * 2, n_seq * H * 4 * dk * pairs),
+            "causal_conv_silu[delta]": (n_tok * C * 4, 0),
+            "causal_conv_silu[parallel]": (n_tok * inner * 4, 0),
+            "delta_scan": (n_tok * (C * 2 + RH * 4 + RH * rdv * 4) + 2 * n_seq * RH * rdk * rdv * 4, 0),
+            "head_norm_act_gate": (n_tok * RH * rdv * 8, 0),
+            "selective_scan": (n_tok * (inner * 8 + N * 4) + 2 * n_seq * inner * N * 4, 0),
+            "gelu_glu": (n_tok * s["ff"] * 6, 0),
         }
         for name, ts in by.items():
             t = statistics.mean(ts)
