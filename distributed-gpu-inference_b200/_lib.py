@@ -270,7 +270,7 @@ MIXER_SIGNATURES = {
                 c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_float, c_float, c_int, c_int,
                 c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p,
                 c_int, c_void_p]),
-    "b200_mixed_prompt_attn_rows_supported": (c_int, [c_int, c_int, c_int, c_int, c_int]),
+    "b200_mixed_prompt_attn_rows_supported": (c_int, [c_int, c_int, c_int, c_int]),
     "b200_qknorm_rotary_append_ext2": (
         c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int, c_float, c_void_p,
                 c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int,

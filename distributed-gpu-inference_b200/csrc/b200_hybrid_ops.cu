@@ -262,8 +262,8 @@ struct AttnArgs {
   int chunk = 0;   // > 0: a position sees only the keys of its own block of `chunk` positions (counted from 0)
   int v_row = 0;   // elements between value rows in v_pool (the value size unless the values are the first columns of wider rows)
   int v_div = 1;   // value head = key head / v_div (several key heads read one value head)
-  int row_heads = 0;   // tensor-core kernel, > 0: a tile is ONE token and its 16 rows are consecutive heads of the `row_heads`
-                       // that share a kv head; H then counts groups of 16 heads (or what is left of a kv head's)
+  int row_heads = 0;   // tensor-core kernel, > 0: a tile is ONE token and its 16 rows are consecutive heads of `row_heads`
+                       // that share one kv head; H then counts groups of 16 heads
   int out_f32 = 0;     // != 0: `out` is fp32 (same strides, in elements) whatever T is; plain outputs only (no turn back)
   int stage_q = 0;     // tensor-core kernel: a warp's 16 query rows are staged in shared memory once (always with row_heads)
   int gate_dim = 0;    // 0: one gate per head (rows of H); the value size: one per output channel (rows of H * dv)
@@ -531,12 +531,14 @@ constexpr int kTcRows = 16;
 constexpr int kTcRawStride = 40;
 
 // EXT: the kernel also knows blocks of positions, values inside wider rows or shared by several key heads, and heads on
-// the rows; layers without any of these run the instantiation that carries none of it.
-template <typename T, int DV8, int HW, bool EXT>
+// the rows; GATED, that gates may be per channel.  Layers without any of these run the instantiation that carries none of it.
+constexpr int kTcPlain = 0, kTcGated = 1, kTcExt = 2;      // kTcExt carries everything
+template <typename T, int DV8, int HW, int MODE>
 __global__ void __launch_bounds__(kTcWarps * 32, (HW == 1 && DV8 <= 16) ? 2 : 1)
 mixed_prompt_attn_kernel(const AttnArgs A, const int32_t* __restrict__ tiles, const float* __restrict__ rot_tab,
                          float* __restrict__ ws, int n_tok, int stages) {
   extern __shared__ __align__(16) unsigned char tc_smem[];
+  constexpr bool EXT = MODE == kTcExt, GATED = MODE != kTcPlain;
   constexpr int HC = kTcWarps * HW;
   constexpr int DVP = DV8 * 8;
   const int row0 = tiles[3 * blockIdx.x], cnt = tiles[3 * blockIdx.x + 1], trow = tiles[3 * blockIdx.x + 2];
@@ -564,10 +566,8 @@ mixed_prompt_attn_kernel(const AttnArgs A, const int32_t* __restrict__ tiles, co
   float* raw = reinterpret_cast<float*>(stage0 + stages * stage_elems);         // [H][16][40]
   float* talk_s = raw + (mixed ? H * kTcRows * kTcRawStride : 0);                               // [HC][H]
   const int RH = EXT ? A.row_heads : 0;
-  // heads on the rows: group h of 16 rows starts at head `head0(h)` and holds `rows_of(h)` of its kv head's heads
-  const int PG = RH ? (RH + 15) / 16 : 1;
-  auto head0 = [&](int h) { return RH ? (h / PG) * RH + 16 * (h % PG) : h; };
-  auto rows_of = [&](int h) { return RH ? min(16, RH - 16 * (h % PG)) : cnt; };
+  auto head0 = [&](int h) { return RH ? 16 * h : h; };                  // the head of a warp's first row, and its rows in use
+  auto rows_of = [&](int h) { return RH ? min(16, RH - 16 * h) : cnt; };
   // a warp's 16 query rows staged once: few resident warps cannot hide the latency of re-reading them for every key tile
   // (heads on the rows: one warp per CTA; wide value layouts: one CTA per SM)
   const bool QS = EXT && A.stage_q;
@@ -796,7 +796,7 @@ mixed_prompt_attn_kernel(const AttnArgs A, const int32_t* __restrict__ tiles, co
       for (int half = 0; half < 2; ++half) {
         const int row = qr + 8 * half;
         if (row >= rows_of(h)) continue;
-        float* dst = RH ? ws + ((static_cast<int64_t>(blockIdx.z) * n_tok + row0) * (RH * G) + head0(h) + row) * (DVP + 2)
+        float* dst = RH ? ws + ((static_cast<int64_t>(blockIdx.z) * n_tok + row0) * RH + head0(h) + row) * (DVP + 2)
                         : ws + ((static_cast<int64_t>(blockIdx.z) * n_tok + row0 + row) * H + h) * (DVP + 2);
         if (qc == 0) {
           dst[0] = m_r[hw][half];
@@ -830,7 +830,7 @@ mixed_prompt_attn_kernel(const AttnArgs A, const int32_t* __restrict__ tiles, co
         } else {
           f = 1.0f / l;
         }
-        if (gate && !A.unrotate && !(EXT && A.gate_dim))
+        if (gate && !A.unrotate && !(GATED && A.gate_dim))
           f *= sigmoid_(Cvt<T>::to_f32(gate[static_cast<int64_t>(RH ? row0 : row0 + row) * A.gate_stride + (RH ? head0(h) + row : h)]));
       }
 #pragma unroll
@@ -850,7 +850,7 @@ mixed_prompt_attn_kernel(const AttnArgs A, const int32_t* __restrict__ tiles, co
         for (int nt = 0; nt < DV8; ++nt) {
           const int c = nt * 8 + qc;
           if (c >= dv) continue;
-          if (EXT && gate && A.gate_dim) {
+          if (GATED && gate && A.gate_dim) {
             const int64_t tok = RH ? row0 : row0 + row;
             O[hw][nt][2 * half] *= gate_at(A, gate, tok, RH ? head0(h) + row : h, c);
             O[hw][nt][2 * half + 1] *= gate_at(A, gate, tok, RH ? head0(h) + row : h, c + 1);
@@ -1465,9 +1465,9 @@ int b200_mixed_prompt_attn_supported(int H, int G, int dk, int dv, int has_talk,
   return tc_plan(H, G, dk, dv, has_talk != 0, same_pool != 0, unrotate != 0, dtype, nullptr) ? 1 : 0;
 }
 
-int b200_mixed_prompt_attn_rows_supported(int H, int G, int dk, int dv, int dtype) {
-  if (H <= 0 || G <= 0 || H % G) return 0;
-  return tc_plan(G * ((H / G + 15) / 16), G, dk, dv, false, false, false, dtype, nullptr, true) ? 1 : 0;
+int b200_mixed_prompt_attn_rows_supported(int H, int dk, int dv, int dtype) {
+  if (H <= 0) return 0;
+  return tc_plan((H + 15) / 16, 1, dk, dv, false, false, false, dtype, nullptr, true) ? 1 : 0;
 }
 
 int b200_mixed_prompt_attn_splits(int n_tiles, int key_tiles, int H, int G, int dk, int dv, int has_talk, int same_pool,
@@ -1507,8 +1507,6 @@ int b200_mixed_prompt_attn_ext(void* out, int64_t out_tok_stride, int64_t out_he
                                const float* value_rot, int interleaved, int H, int G, int dk, int dv, int v_row, int v_div,
                                int heads_as_rows, int out_f32, int block_size, int n_splits, float* workspace, int dtype,
                                void* stream) {
-  if (heads_as_rows && (G != 1 || gate))
-    return fail(B200_EINVAL, "b200_mixed_prompt_attn: heads as rows need one kv head and no mixing, gate or value rotation");
   return b200_mixed_prompt_attn_ext2(out, out_tok_stride, out_head_stride, q, q_tok_stride, q_head_stride, gate, gate_stride,
                                      0, k_pool, v_pool, block_tables, table_stride, tiles, n_tiles, tok_pos, n_tok, talk,
                                      sink, scale, softcap, window, keep_first, chunk, value_rot, interleaved, H, G, dk, dv,
@@ -1527,12 +1525,12 @@ int b200_mixed_prompt_attn_ext2(void* out, int64_t out_tok_stride, int64_t out_h
   if (out_f32 && value_rot) return fail(B200_EINVAL, "b200_mixed_prompt_attn: fp32 outputs are not turned back");
   if (chunk < 0 || v_row < dv || v_row % 8 || v_div < 1 || G % v_div)
     return fail(B200_EINVAL, "b200_mixed_prompt_attn: bad mask or value layout");
-  if (heads_as_rows && (G <= 0 || H % G || v_div != 1 || talk || value_rot))
-    return fail(B200_EINVAL, "b200_mixed_prompt_attn: heads as rows allow no mixing, shared values or value rotation");
+  if (heads_as_rows && (G != 1 || talk || value_rot))
+    return fail(B200_EINVAL, "b200_mixed_prompt_attn: heads as rows need one kv head and no mixing or value rotation");
   if (heads_as_rows && (!aligned16(q) || ((q_tok_stride | q_head_stride) & 7)))
     return fail(B200_ESHAPE, "b200_mixed_prompt_attn: heads as rows need 16-byte aligned query rows");
   const int H_real = H;
-  if (heads_as_rows) H = G * ((H / G + 15) / 16);      // the kernel's heads are groups of up to 16 rows of one kv head
+  if (heads_as_rows) H = (H + 15) / 16;      // the kernel's heads are groups of 16 rows
   if (n_tiles < 0 || n_tok < 0 || H <= 0 || G <= 0 || H % G || dk <= 0 || dv <= 0 || block_size <= 0 || n_splits < 1 ||
       n_splits > 64)
     return fail(B200_EINVAL, "b200_mixed_prompt_attn: bad sizes");
@@ -1545,7 +1543,7 @@ int b200_mixed_prompt_attn_ext2(void* out, int64_t out_tok_stride, int64_t out_h
   // query rows are staged where few warps are resident anyway: heads on the rows, and the widest value layout (one CTA
   // per SM by its registers) when its rows allow 16-byte reads
   const bool q_ok = aligned16(q) && !((q_tok_stride | q_head_stride) & 7);
-  const bool ext_call = chunk > 0 || v_div > 1 || v_row != dv || heads_as_rows || out_f32 || gate_per_channel;
+  const bool ext_call = chunk > 0 || v_div > 1 || v_row != dv || heads_as_rows || out_f32;
   bool stage_q = heads_as_rows || (ext_call && dv > 128 && q_ok);
   if (stage_q && !heads_as_rows && !tc_plan(H, G, dk, dv, talk != nullptr, k_pool == v_pool, value_rot != nullptr, dtype, &plan, true))
     stage_q = false;
@@ -1553,7 +1551,7 @@ int b200_mixed_prompt_attn_ext2(void* out, int64_t out_tok_stride, int64_t out_h
     return fail(B200_ESHAPE, "b200_mixed_prompt_attn: sizes off the tensor-core grid (dk %d, dv %d)", dk, dv);
   AttnArgs A{out, out_tok_stride, out_head_stride, q, q_tok_stride, q_head_stride, gate, gate_stride, k_pool, v_pool,
              block_tables, table_stride, nullptr, tok_pos, talk, sink, scale, window, keep_first, value_rot != nullptr,
-             interleaved, 0.0, H, G, dk, dv, block_size, softcap, chunk, v_row, v_div, heads_as_rows ? H_real / G : 0,
+             interleaved, 0.0, H, G, dk, dv, block_size, softcap, chunk, v_row, v_div, heads_as_rows ? H_real : 0,
              out_f32, stage_q ? 1 : 0, gate_per_channel ? dv : 0};
   const dim3 grid(n_tiles, (H + kTcWarps * plan.hw - 1) / (kTcWarps * plan.hw), n_splits);
   return hybrid_by_dtype(dtype, "b200_mixed_prompt_attn", [&](auto* tag) {
@@ -1568,20 +1566,17 @@ int b200_mixed_prompt_attn_ext2(void* out, int64_t out_tok_stride, int64_t out_h
         cudaFuncSetAttribute(kern, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
         kern<<<grid, kTcWarps * 32, plan.smem, s>>>(A, tiles, value_rot, workspace, n_tok, plan.stages);
       };
-      const bool ext = ext_call;
-      if (ext) {
-        if (plan.dv8 == 8 && plan.hw == 1) launch(mixed_prompt_attn_kernel<T, 8, 1, true>);
-        else if (plan.dv8 == 8) launch(mixed_prompt_attn_kernel<T, 8, 2, true>);
-        else if (plan.dv8 == 16 && plan.hw == 1) launch(mixed_prompt_attn_kernel<T, 16, 1, true>);
-        else if (plan.dv8 == 16) launch(mixed_prompt_attn_kernel<T, 16, 2, true>);
-        else launch(mixed_prompt_attn_kernel<T, 32, 1, true>);
-      } else {
-        if (plan.dv8 == 8 && plan.hw == 1) launch(mixed_prompt_attn_kernel<T, 8, 1, false>);
-        else if (plan.dv8 == 8) launch(mixed_prompt_attn_kernel<T, 8, 2, false>);
-        else if (plan.dv8 == 16 && plan.hw == 1) launch(mixed_prompt_attn_kernel<T, 16, 1, false>);
-        else if (plan.dv8 == 16) launch(mixed_prompt_attn_kernel<T, 16, 2, false>);
-        else launch(mixed_prompt_attn_kernel<T, 32, 1, false>);
-      }
+      auto pick = [&](auto mode) {
+        constexpr int M = decltype(mode)::value;
+        if (plan.dv8 == 8 && plan.hw == 1) launch(mixed_prompt_attn_kernel<T, 8, 1, M>);
+        else if (plan.dv8 == 8) launch(mixed_prompt_attn_kernel<T, 8, 2, M>);
+        else if (plan.dv8 == 16 && plan.hw == 1) launch(mixed_prompt_attn_kernel<T, 16, 1, M>);
+        else if (plan.dv8 == 16) launch(mixed_prompt_attn_kernel<T, 16, 2, M>);
+        else launch(mixed_prompt_attn_kernel<T, 32, 1, M>);
+      };
+      if (ext_call) pick(std::integral_constant<int, kTcExt>{});
+      else if (gate_per_channel) pick(std::integral_constant<int, kTcGated>{});
+      else pick(std::integral_constant<int, kTcPlain>{});
       int rc = check_launch("b200_mixed_prompt_attn");
       if (rc != 0 || n_splits == 1) return rc;
       // every packed row belongs to exactly one tile, so the merge runs over all rows

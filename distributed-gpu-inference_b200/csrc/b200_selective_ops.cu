@@ -231,19 +231,71 @@ struct SelArgs {
   float* state;                       // [slots][I][N]
   const SelSeq* seqs;
   int I, N, lg;                       // lg: log2 of the lanes that share a channel
-  int vec;                            // rows of x, dt and z may be copied in 16-byte pieces
+  int vec;                            // rows of x, dt and z may be copied in 16-byte pieces and out written in pairs
+  int vec_bc;                         // rows of B and C may be copied in 16-byte pieces
 };
 
-// S <- exp(dt A) S + w.  16-bit models: A2 = A log2(e) and the hardware's exp2 instruction.  fp32: A2 = A and S + (exp(dt A) - 1) S:
-// a factor just below one would be rounded the same way for thousands of tokens, its distance to one is not.
+// Step sizes and gates of 16-bit models use the hardware's exponential and reciprocal (relative errors of a few 1e-7).
+// softplus(z) = max(z, 0) + log(1 + u), u = exp(-|z|), with log(1 + u) = 2 artanh(r), r = u / (2 + u) <= 1/3, and the Taylor
+// series artanh(r) = r (1 + r^2/3 + r^4/5 + ...), cut after r^12 / 13 (relative remainder below 2e-8): accurate for small u too.
 template <typename T>
-__device__ __forceinline__ float decayed(float S, float dt, float a2, float w) {
+__device__ __forceinline__ float step_of(float z) {
   if constexpr (sizeof(T) == 4) {
-    return S + fmaf(expm1f(dt * a2), S, w);
+    return softplus_f(z);
   } else {
-    float r;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(dt * a2));
-    return fmaf(r, S, w);
+    const float u = __expf(-fabsf(z)), r = __fdividef(u, 2.0f + u), q = r * r;
+    float p = fmaf(q, 1.0f / 13.0f, 1.0f / 11.0f);
+    p = fmaf(p, q, 1.0f / 9.0f);
+    p = fmaf(p, q, 1.0f / 7.0f);
+    p = fmaf(p, q, 1.0f / 5.0f);
+    p = fmaf(p, q, 1.0f / 3.0f);
+    p = fmaf(p, q, 1.0f);
+    return fmaxf(z, 0.f) + 2.0f * r * p;
+  }
+}
+template <typename T>
+__device__ __forceinline__ float gate_of(float z) {
+  if constexpr (sizeof(T) == 4) return silu_f(z);
+  else return __fdividef(z, 1.0f + __expf(-z));
+}
+
+// Two fp32 numbers in one 64-bit register: sm_100 multiplies and adds both with one instruction.
+using f32x2 = unsigned long long;
+__device__ __forceinline__ f32x2 pack2(float lo, float hi) {
+  f32x2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ void unpack2(f32x2 v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ f32x2 mul2(f32x2 a, f32x2 b) {
+  f32x2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ f32x2 fma2(f32x2 a, f32x2 b, f32x2 c) {
+  f32x2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ float exp2_hw(float x) {
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
+
+// S <- exp(dt A) S + w for two states.  16-bit models: A2 = A log2(e) and the hardware's exp2 instruction.  fp32: A2 = A and
+// S + (exp(dt A) - 1) S: a factor just below one would be rounded the same way for thousands of tokens, its distance to one is not.
+template <typename T>
+__device__ __forceinline__ f32x2 decayed(f32x2 S, f32x2 dt, f32x2 a2, f32x2 w) {
+  float x, y;
+  unpack2(mul2(dt, a2), x, y);
+  if constexpr (sizeof(T) == 4) {
+    float s, t;
+    unpack2(fma2(pack2(expm1f(x), expm1f(y)), S, w), x, y);
+    unpack2(S, s, t);
+    return pack2(s + x, t + y);
+  } else {
+    return fma2(pack2(exp2_hw(x), exp2_hw(y)), S, w);
   }
 }
 
@@ -254,15 +306,16 @@ __device__ __forceinline__ void sel_copy16(void* dst, const void* src, bool vali
 }
 
 // One CTA (128 threads) per (sequence, 128 / L channels), L = 2^lg adjacent lanes per channel, NPT states each in registers for
-// the whole portion.  32 tokens are staged at a time: the rows of x, dt and the gate arrive by cp.async one stage ahead; step
-// sizes (one softplus per token and channel) and B, C in fp32 are formed once per stage; the read-outs leave gated.
+// the whole portion.  32 tokens are staged at a time: their rows arrive by cp.async one stage ahead; step sizes (one softplus per
+// token and channel) and B, C in fp32 are formed once per stage; the read-outs leave gated.  Four tokens are computed together:
+// only the four multiply-adds of a state depend on each other, and the lanes of a channel sum four read-outs in one butterfly.
 constexpr int kSelNT = 128;
 constexpr int kSelTok = 32;
 
 template <typename T>
-inline size_t sel_smem(int ch, int np) {
+inline size_t sel_smem(int ch, int np, int n) {
   return sizeof(float) * kSelTok * (2 * static_cast<size_t>(ch) + 2 * static_cast<size_t>(np)) +
-         2 * 3 * kSelTok * static_cast<size_t>(ch) * sizeof(T);
+         2 * kSelTok * (3 * static_cast<size_t>(ch) + 2 * static_cast<size_t>(n)) * sizeof(T);
 }
 
 template <typename T, int NPT>
@@ -271,11 +324,12 @@ selective_scan_kernel(const SelArgs A) {
   extern __shared__ __align__(16) unsigned char sel_raw[];
   const SelSeq sq = A.seqs[blockIdx.y];
   if (sq.count <= 0) return;
-  const int tid = threadIdx.x, lg = A.lg, L = 1 << lg, CH = kSelNT >> lg, NP = NPT << lg;
+  const int tid = threadIdx.x, lg = A.lg, L = 1 << lg, lgc = 7 - lg, CH = 1 << lgc, NP = NPT << lg;
   const int I = A.I, N = A.N, c0 = blockIdx.x * CH, nch = min(CH, I - c0);
   float2* ds = reinterpret_cast<float2*>(sel_raw);                       // (dt, dt x) [tok][CH]; later (read-out, -)
   float* bc = reinterpret_cast<float*>(ds + kSelTok * CH);               // B | C, [tok][2 NP]
-  T* raw = reinterpret_cast<T*>(bc + kSelTok * 2 * NP);                  // [2 stages][x, dt, z][tok][CH]
+  T* raw = reinterpret_cast<T*>(bc + kSelTok * 2 * NP);                  // [2 stages]: [x, dt, z][tok][CH], [B, C][tok][N]
+  const int stage_elems = kSelTok * (3 * CH + 2 * N);
   const int cl = tid >> lg, sub = tid & (L - 1), ch = c0 + cl;
   const bool has = cl < nch;
   const T* xp = static_cast<const T*>(A.x) + static_cast<int64_t>(sq.tok0) * A.x_stride + c0;
@@ -285,25 +339,29 @@ selective_scan_kernel(const SelArgs A) {
   const T* cp = static_cast<const T*>(A.c) + static_cast<int64_t>(sq.tok0) * A.bc_stride;
   T* op = static_cast<T*>(A.out) + static_cast<int64_t>(sq.tok0) * A.out_stride + c0;
   float* st = A.state + (static_cast<int64_t>(sq.slot) * I + ch) * N;
+  // the channels a thread converts and stores never change from stage to stage: two neighbours (vec) or one
+  const int cv = A.vec ? (tid & (CH / 2 - 1)) * 2 : tid & (CH - 1);
+  const int tv = A.vec ? tid >> (lgc - 1) : tid >> lgc, tstep = A.vec ? kSelNT >> (lgc - 1) : kSelNT >> lgc;
+  const bool cok = cv < nch;
+  const float bias0 = cok ? A.dt_bias[c0 + cv] : 0.f, bias1 = cok && A.vec ? A.dt_bias[c0 + cv + 1] : 0.f;
+  const float skip0 = cok ? A.skip[c0 + cv] : 0.f, skip1 = cok && A.vec ? A.skip[c0 + cv + 1] : 0.f;
 
   auto load_stage = [&](int t0, int buf) {
-    T* dst = raw + buf * 3 * kSelTok * CH;
+    T* dst = raw + buf * stage_elems;
     const int nt = min(kSelTok, sq.count - t0);
+    constexpr int E = 16 / sizeof(T), LE = sizeof(T) == 4 ? 2 : 3;
     if (A.vec) {
-      constexpr int E = 16 / sizeof(T);
-      const int pieces = CH / E;
-      for (int e = tid; e < 3 * kSelTok * pieces; e += kSelNT) {
-        const int which = e / (kSelTok * pieces), r = e - which * kSelTok * pieces;
-        const int t = r / pieces, c = (r - t * pieces) * E;
+      const int lp = lgc - LE;                                           // log2 of the pieces of a row
+      for (int e = tid; e < (3 * kSelTok) << lp; e += kSelNT) {
+        const int row = e >> lp, which = row / kSelTok, t = row & (kSelTok - 1), c = (e & ((1 << lp) - 1)) * E;
         const bool ok = t < nt && c < nch;
         const T* src = which == 0 ? xp : (which == 1 ? dp : zp);
         const int64_t stride = which == 0 ? A.x_stride : (which == 1 ? A.dt_stride : A.z_stride);
-        sel_copy16(dst + (which * kSelTok + t) * CH + c, ok ? src + static_cast<int64_t>(t0 + t) * stride + c : src, ok);
+        sel_copy16(dst + row * CH + c, ok ? src + static_cast<int64_t>(t0 + t) * stride + c : src, ok);
       }
-      asm volatile("cp.async.commit_group;" ::: "memory");
     } else {
       for (int e = tid; e < kSelTok * CH; e += kSelNT) {
-        const int t = e / CH, c = e - t * CH;
+        const int t = e >> lgc, c = e & (CH - 1);
         if (t < nt && c < nch) {
           dst[t * CH + c] = xp[static_cast<int64_t>(t0 + t) * A.x_stride + c];
           dst[(kSelTok + t) * CH + c] = dp[static_cast<int64_t>(t0 + t) * A.dt_stride + c];
@@ -311,98 +369,147 @@ selective_scan_kernel(const SelArgs A) {
         }
       }
     }
+    dst += 3 * kSelTok * CH;
+    const int t = tid >> 2;                                              // four threads per row of B and C
+    if (A.vec_bc) {
+      for (int n = (tid & 3) * E; n < 2 * N; n += 4 * E) {
+        const T* src = n < N ? bp + n : cp + n - N;
+        sel_copy16(dst + t * 2 * N + n, t < nt ? src + static_cast<int64_t>(t0 + t) * A.bc_stride : src, t < nt);
+      }
+    } else if (t < nt) {
+      for (int n = tid & 3; n < 2 * N; n += 4) dst[t * 2 * N + n] = (n < N ? bp + n : cp + n - N)[static_cast<int64_t>(t0 + t) * A.bc_stride];
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
   };
   load_stage(0, 0);
-  float S[NPT], a2[NPT];
+  f32x2 S[NPT / 2], a2[NPT / 2];
 #pragma unroll
-  for (int j = 0; j < NPT; ++j) {
-    const int n = sub * NPT + j;
-    const bool ok = has && n < N;
-    S[j] = (ok && !sq.fresh) ? st[n] : 0.f;
-    a2[j] = ok ? -expf(A.a_log[static_cast<int64_t>(ch) * N + n]) * (sizeof(T) == 4 ? 1.0f : 1.4426950408889634f) : 0.f;
+  for (int j = 0; j < NPT; j += 2) {
+    float s[2], a[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int n = sub * NPT + j + i;
+      const bool ok = has && n < N;
+      s[i] = (ok && !sq.fresh) ? st[n] : 0.f;
+      a[i] = ok ? -expf(A.a_log[static_cast<int64_t>(ch) * N + n]) * (sizeof(T) == 4 ? 1.0f : 1.4426950408889634f) : 0.f;
+    }
+    S[j / 2] = pack2(s[0], s[1]);
+    a2[j / 2] = pack2(a[0], a[1]);
   }
   for (int t0 = 0, buf = 0; t0 < sq.count; t0 += kSelTok, buf ^= 1) {
-    const int nt = min(kSelTok, sq.count - t0);
-    const T* rx = raw + buf * 3 * kSelTok * CH;
+    const int nt = min(kSelTok, sq.count - t0), nt4 = (nt + 3) & ~3;     // up to three tokens of padding: dt = 0 leaves the state
+    const T* rx = raw + buf * stage_elems;
     const T* rd = rx + kSelTok * CH;
     const T* rz = rd + kSelTok * CH;
-    // B and C of the stage (their slots were last read before the barrier that ended the previous stage)
-    for (int e = tid; e < nt * NP; e += kSelNT) {
-      const int t = e / NP, n = e - t * NP;
-      bc[t * 2 * NP + n] = n < N ? Cvt<T>::to_f32(bp[static_cast<int64_t>(t0 + t) * A.bc_stride + n]) : 0.f;
-      bc[t * 2 * NP + NP + n] = n < N ? Cvt<T>::to_f32(cp[static_cast<int64_t>(t0 + t) * A.bc_stride + n]) : 0.f;
-    }
+    const T* rbc = rz + kSelTok * CH;
     asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
     if (t0 + kSelTok < sq.count) load_stage(t0 + kSelTok, buf ^ 1);
-    for (int e = tid; e < nt * CH; e += kSelNT) {
-      const int c = e % CH;
-      if (c < nch) {
-        const float dt = softplus_f(Cvt<T>::to_f32(rd[e]) + A.dt_bias[c0 + c]);
-        ds[e] = make_float2(dt, dt * Cvt<T>::to_f32(rx[e]));
+#pragma unroll 4
+    for (int t = tv; t < nt4; t += tstep) {
+      const int e = t * CH + cv;
+      const bool ok = cok && t < nt;
+      const float da = ok ? step_of<T>(Cvt<T>::to_f32(rd[e]) + bias0) : 0.f;
+      const float xa = ok ? Cvt<T>::to_f32(rx[e]) : 0.f;
+      if (A.vec) {
+        const float db = ok ? step_of<T>(Cvt<T>::to_f32(rd[e + 1]) + bias1) : 0.f;
+        const float xb = ok ? Cvt<T>::to_f32(rx[e + 1]) : 0.f;
+        *reinterpret_cast<float4*>(ds + e) = make_float4(da, da * xa, db, db * xb);
       } else {
-        ds[e] = make_float2(0.f, 0.f);
+        ds[e] = make_float2(da, da * xa);
       }
+    }
+    {
+      const int t = tid >> 2;
+      if (t < nt4)
+        for (int n = tid & 3; n < NP; n += 4) {
+          const bool ok = t < nt && n < N;
+          bc[t * 2 * NP + n] = ok ? Cvt<T>::to_f32(rbc[t * 2 * N + n]) : 0.f;
+          bc[t * 2 * NP + NP + n] = ok ? Cvt<T>::to_f32(rbc[t * 2 * N + N + n]) : 0.f;
+        }
     }
     __syncthreads();
     const float* bt = bc + sub * NPT;
-#pragma unroll 2
-    for (int t = 0; t < nt; ++t) {
-      const float2 d = ds[t * CH + cl];
-      float B[NPT], C[NPT];
-      if constexpr (NPT % 4 == 0) {
+    for (int t = 0; t < nt4; t += 4) {
+      float2 d[4];
+      float y[4];
 #pragma unroll
-        for (int j = 0; j < NPT; j += 4) {
-          *reinterpret_cast<float4*>(B + j) = *reinterpret_cast<const float4*>(bt + t * 2 * NP + j);
-          *reinterpret_cast<float4*>(C + j) = *reinterpret_cast<const float4*>(bt + t * 2 * NP + NP + j);
-        }
-      } else {
+      for (int u = 0; u < 4; ++u) d[u] = ds[(t + u) * CH + cl];
 #pragma unroll
-        for (int j = 0; j < NPT; j += 2) {
-          *reinterpret_cast<float2*>(B + j) = *reinterpret_cast<const float2*>(bt + t * 2 * NP + j);
-          *reinterpret_cast<float2*>(C + j) = *reinterpret_cast<const float2*>(bt + t * 2 * NP + NP + j);
-        }
-      }
-      float y0 = 0.f, y1 = 0.f;
+      for (int u = 0; u < 4; ++u) {
+        const float* row = bt + (t + u) * 2 * NP;
+        f32x2 B[NPT / 2], C[NPT / 2];
+        if constexpr (NPT % 4 == 0) {
 #pragma unroll
-      for (int j = 0; j < NPT; j += 2) {
-        S[j] = decayed<T>(S[j], d.x, a2[j], d.y * B[j]);
-        y0 = fmaf(S[j], C[j], y0);
-        S[j + 1] = decayed<T>(S[j + 1], d.x, a2[j + 1], d.y * B[j + 1]);
-        y1 = fmaf(S[j + 1], C[j + 1], y1);
-      }
-      float y = y0 + y1;
-      if (lg > 0) {
-        y += __shfl_xor_sync(0xffffffffu, y, 1);
-        if (lg > 1) {
-          y += __shfl_xor_sync(0xffffffffu, y, 2);
-          if (lg > 2) {
-            y += __shfl_xor_sync(0xffffffffu, y, 4);
-            if (lg > 3) {
-              y += __shfl_xor_sync(0xffffffffu, y, 8);
-              if (lg > 4) y += __shfl_xor_sync(0xffffffffu, y, 16);
-            }
+          for (int j = 0; j < NPT; j += 4) {
+            const ulonglong2 b2 = *reinterpret_cast<const ulonglong2*>(row + j), c2 = *reinterpret_cast<const ulonglong2*>(row + NP + j);
+            B[j / 2] = b2.x;
+            B[j / 2 + 1] = b2.y;
+            C[j / 2] = c2.x;
+            C[j / 2 + 1] = c2.y;
+          }
+        } else {
+#pragma unroll
+          for (int j = 0; j < NPT; j += 2) {
+            B[j / 2] = *reinterpret_cast<const f32x2*>(row + j);
+            C[j / 2] = *reinterpret_cast<const f32x2*>(row + NP + j);
           }
         }
+        const f32x2 dt2 = pack2(d[u].x, d[u].x), dx2 = pack2(d[u].y, d[u].y);
+        f32x2 acc = pack2(0.f, 0.f);
+#pragma unroll
+        for (int j = 0; j < NPT / 2; ++j) {
+          S[j] = decayed<T>(S[j], dt2, a2[j], mul2(dx2, B[j]));
+          acc = fma2(S[j], C[j], acc);
+        }
+        float y0, y1;
+        unpack2(acc, y0, y1);
+        y[u] = y0 + y1;
       }
-      // the channel's lanes have read (dt, dt x) of this token: they are in one warp, and the shuffles (or nothing, when a lane
-      // is alone) come after their reads
-      if (sub == 0) ds[t * CH + cl].x = y;
+      // the channel's lanes have read (dt, dt x) of these tokens: they are in one warp, and the shuffles come after their reads
+      if (lg == 0) {
+#pragma unroll
+        for (int u = 0; u < 4; ++u) ds[(t + u) * CH + cl].x = y[u];
+      } else {
+        const bool odd = sub & 1;
+        float k0 = (odd ? y[2] : y[0]) + __shfl_xor_sync(0xffffffffu, odd ? y[0] : y[2], 1);
+        float k1 = (odd ? y[3] : y[1]) + __shfl_xor_sync(0xffffffffu, odd ? y[1] : y[3], 1);
+        const int tk = t + (odd ? 2 : 0);
+        if (lg == 1) {
+          ds[tk * CH + cl].x = k0;
+          ds[(tk + 1) * CH + cl].x = k1;
+        } else {
+          const bool hi = sub & 2;
+          float k = (hi ? k1 : k0) + __shfl_xor_sync(0xffffffffu, hi ? k0 : k1, 2);
+          for (int o = 4; o < L; o <<= 1) k += __shfl_xor_sync(0xffffffffu, k, o);
+          if (sub < 4) ds[(tk + (hi ? 1 : 0)) * CH + cl].x = k;
+        }
+      }
     }
     __syncthreads();
-    for (int e = tid; e < nt * CH; e += kSelNT) {
-      const int t = e / CH, c = e - t * CH;
-      if (c < nch) {
-        const float y = fmaf(A.skip[c0 + c], Cvt<T>::to_f32(rx[e]), ds[e].x);
-        op[static_cast<int64_t>(t0 + t) * A.out_stride + c] = Cvt<T>::from_f32(A.gain * y * silu_f(Cvt<T>::to_f32(rz[e])));
+    if (cok)
+#pragma unroll 4
+      for (int t = tv; t < nt; t += tstep) {
+        const int e = t * CH + cv;
+        T* dst = op + static_cast<int64_t>(t0 + t) * A.out_stride + cv;
+        const float ya = A.gain * fmaf(skip0, Cvt<T>::to_f32(rx[e]), ds[e].x) * gate_of<T>(Cvt<T>::to_f32(rz[e]));
+        if (A.vec) {
+          const float yb = A.gain * fmaf(skip1, Cvt<T>::to_f32(rx[e + 1]), ds[e + 1].x) * gate_of<T>(Cvt<T>::to_f32(rz[e + 1]));
+          struct alignas(2 * sizeof(T)) Pair { T a, b; };
+          *reinterpret_cast<Pair*>(dst) = Pair{Cvt<T>::from_f32(ya), Cvt<T>::from_f32(yb)};
+        } else {
+          *dst = Cvt<T>::from_f32(ya);
+        }
       }
-    }
     __syncthreads();
   }
 #pragma unroll
-  for (int j = 0; j < NPT; ++j) {
+  for (int j = 0; j < NPT; j += 2) {
+    float lo, hi;
+    unpack2(S[j / 2], lo, hi);
     const int n = sub * NPT + j;
-    if (has && n < N) st[n] = S[j];
+    if (has && n < N) st[n] = lo;
+    if (has && n + 1 < N) st[n + 1] = hi;
   }
 }
 
@@ -521,7 +628,7 @@ int b200_selective_scan(void* out, int64_t out_stride, const void* x, int64_t x_
                         const float* skip, const void* z, int64_t z_stride, float gain, float* state, const int32_t* seqs,
                         int n_seqs, int inner, int n_state, int dtype, void* stream) {
   SelArgs A{out, out_stride, x, x_stride, dt, dt_stride, dt_bias, a_log, b, c, bc_stride, skip, z, z_stride, gain, state,
-            reinterpret_cast<const SelSeq*>(seqs), inner, n_state, 0, 0};
+            reinterpret_cast<const SelSeq*>(seqs), inner, n_state, 0, 0, 0};
   if (const int rc = sel_check("b200_selective_scan", A, n_seqs)) return rc;
   if (n_state > 256) return fail(B200_ESHAPE, "b200_selective_scan: %d states per channel beyond 256", n_state);
   if (n_seqs == 0) return 0;
@@ -529,7 +636,7 @@ int b200_selective_scan(void* out, int64_t out_stride, const void* x, int64_t x_
   int lg = 0;
   while ((8 << lg) < n_state) ++lg;
   auto warps = [&](int l) { return static_cast<int64_t>(n_seqs) * ((static_cast<int64_t>(inner) << l) + 127) / 128 * 4; };
-  while (lg < 5 && warps(lg) < kNumSMs * 6 && ((n_state + (1 << lg) - 1) >> lg) > 2) ++lg;
+  while (lg < 5 && warps(lg) < kNumSMs * 8 && ((n_state + (1 << lg) - 1) >> lg) > 2) ++lg;
   A.lg = lg;
   const int npt = (n_state + (1 << lg) - 1) >> lg;
   const int ch = kSelNT >> lg;
@@ -537,9 +644,10 @@ int b200_selective_scan(void* out, int64_t out_stride, const void* x, int64_t x_
     using T = std::remove_pointer_t<decltype(tag)>;
     constexpr int E = 16 / sizeof(T);
     A.vec = ch % E == 0 && inner % E == 0 && x_stride % E == 0 && dt_stride % E == 0 && z_stride % E == 0 && aligned16(x) &&
-            aligned16(dt) && aligned16(z);
+            aligned16(dt) && aligned16(z) && out_stride % 2 == 0 && reinterpret_cast<uintptr_t>(out) % (2 * sizeof(T)) == 0;
+    A.vec_bc = n_state % E == 0 && bc_stride % E == 0 && aligned16(b) && aligned16(c);
     auto launch = [&](auto kern, int per_lane) {
-      const size_t smem = sel_smem<T>(ch, per_lane << lg);
+      const size_t smem = sel_smem<T>(ch, per_lane << lg, n_state);
       if (smem > 48 * 1024) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
       kern<<<dim3((inner + ch - 1) / ch, n_seqs), kSelNT, smem, static_cast<cudaStream_t>(stream)>>>(A);
     };
@@ -556,7 +664,7 @@ int b200_selective_step(void* out, int64_t out_stride, const void* x, int64_t x_
                         const float* skip, const void* z, int64_t z_stride, float gain, float* state, const int32_t* seqs,
                         int n_seqs, int inner, int n_state, int dtype, void* stream) {
   SelArgs A{out, out_stride, x, x_stride, dt, dt_stride, dt_bias, a_log, b, c, bc_stride, skip, z, z_stride, gain, state,
-            reinterpret_cast<const SelSeq*>(seqs), inner, n_state, 0, 0};
+            reinterpret_cast<const SelSeq*>(seqs), inner, n_state, 0, 0, 0};
   if (const int rc = sel_check("b200_selective_step", A, n_seqs)) return rc;
   if (n_seqs == 0) return 0;
   const int per = n_state % 4 == 0 ? n_state / 4 : n_state;      // pieces of a channel's state

@@ -460,9 +460,9 @@ def mixed_prompt_attention_supported(H: int, G: int, dk: int, dv: int, has_talk:
                                                          int(unrotate), DTYPE_ID[dtype]))
 
 
-def heads_as_rows_supported(H: int, G: int, dk: int, dv: int, dtype: torch.dtype) -> bool:
-    """Whether ``mixed_prompt_attention(heads_as_rows=True)`` takes this head layout."""
-    return bool(_lib_().b200_mixed_prompt_attn_rows_supported(int(H), int(G), int(dk), int(dv), DTYPE_ID[dtype]))
+def heads_as_rows_supported(H: int, dk: int, dv: int, dtype: torch.dtype) -> bool:
+    """Whether ``mixed_prompt_attention(heads_as_rows=True)`` takes ``H`` heads over one kv head."""
+    return bool(_lib_().b200_mixed_prompt_attn_rows_supported(int(H), int(dk), int(dv), DTYPE_ID[dtype]))
 
 
 PROMPT_TILE_TOKENS = 16     # tokens of one sequence a CTA of ``mixed_prompt_attention`` serves
@@ -481,9 +481,9 @@ def mixed_prompt_attention(out: torch.Tensor, q: torch.Tensor, k_pool: torch.Ten
     tokens of one sequence each, together covering every row of ``q``; ``value_rot``: the table ``rotary_kv_append``
     returned for this step's tokens; ``max_context``: the longest context of the step (a hint: steps of few tokens over
     long contexts divide the keys over several CTAs and merge); ``chunk``, ``value_width`` and ``value_div`` as in
-    ``mixed_paged_attention``, as are the kinds of ``gate``.  ``heads_as_rows`` (steps of single tokens, no talk / value_rot /
-    value_div; see ``heads_as_rows_supported``): the 16 rows of a tensor-core tile are up to 16 query heads of one token that
-    share a kv head instead of 16 tokens of one head."""
+    ``mixed_paged_attention``, as are the kinds of ``gate``.  ``heads_as_rows`` (steps of single tokens over one kv head,
+    no talk / value_rot; see ``heads_as_rows_supported``): the 16 rows of a tensor-core tile are 16 query heads of one token
+    instead of 16 tokens of one head."""
     _need_cuda(out, q, k_pool, v_pool, block_tables, tiles, tok_pos)
     nb, G, bs, dk = k_pool.shape
     dv, v_row = _value_layout(k_pool, v_pool, value_width, value_div)
@@ -502,14 +502,13 @@ def mixed_prompt_attention(out: torch.Tensor, q: torch.Tensor, k_pool: torch.Ten
                                   or not value_rot.is_contiguous()):
         raise ValueError("value_rot must be contiguous fp32 [n, dv // 2, 2]")
     per_channel = _gate_kind(gate, n, H, dv, q.dtype)
-    if heads_as_rows and (H % G or talk is not None or value_rot is not None or value_div != 1):
-        raise ValueError("heads_as_rows goes with no talk, value_rot or value_div")
-    rows_heads = G * ((H // G + 15) // 16) if heads_as_rows else H
+    if heads_as_rows and (G != 1 or talk is not None or value_rot is not None):
+        raise ValueError("heads_as_rows needs one kv head and no talk or value_rot")
     lib = _lib_()
     seen = min(max_context, window + keep_first + PROMPT_TILE_TOKENS) if window > 0 else max_context
     if chunk > 0:
         seen = min(seen, chunk + PROMPT_TILE_TOKENS)
-    splits = lib.b200_mixed_prompt_attn_splits(tiles.shape[0], (seen + 31) // 32, rows_heads, G,
+    splits = lib.b200_mixed_prompt_attn_splits(tiles.shape[0], (seen + 31) // 32, (H + 15) // 16 if heads_as_rows else H, G,
                                                dk, dv, int(talk is not None),
                                                int(k_pool.data_ptr() == v_pool.data_ptr()), int(value_rot is not None),
                                                DTYPE_ID[q.dtype]) if max_context > 0 else 1

@@ -46,6 +46,7 @@ from .fibirax_layer import wavelength_scaled_frequencies
 from .paged_layer import RaggedLayerCache
 from .petipel_layer import _param
 from .sanesun_layer import UNIT_NORM_EPS, PlainRMSNorm, ScaledFloatEmbedding, _pad8
+from .vatazen_layer import LatentRotaryAttention
 from .worker.distributed.model_shard import ModelShard
 from .zuderax_layer import ScaledHead, _fused
 
@@ -182,8 +183,8 @@ class KeyValueSelectiveMixer(nn.Module):
         self.w_out = _param(w_out, device, dtype)
         self.tensor_cores = mixer_ops.mixed_prompt_attention_supported(self.H, self.G, self.dk, self.dk, False, False, False,
                                                                        self.w_in.dtype)
-        self.rows = (self.tensor_cores and self.H > self.G and
-                     mixer_ops.heads_as_rows_supported(self.H, self.G, self.dk, self.dk, self.w_in.dtype))
+        self.rows = (self.tensor_cores and self.G == 1 and self.H >= LatentRotaryAttention.HEADS_AS_ROWS_FROM and
+                     mixer_ops.heads_as_rows_supported(self.H, self.dk, self.dk, self.w_in.dtype))
 
     def forward(self, h: torch.Tensor, cache: RaggedLayerCache) -> torch.Tensor:
         st, n, c = cache.state, h.shape[0], self.cuts

@@ -195,7 +195,7 @@ int b200_mixed_prompt_attn(void* out, int64_t out_tok_stride, int64_t out_head_s
                            void* stream);
 
 /* b200_mixed_prompt_attn with chunk, v_row and v_div as in b200_mixed_paged_attn_ext (v_row a multiple of 8).
- * heads_as_rows != 0 (steps of single tokens over ONE kv head, G == 1, no talk / gate / value_rot): every tile is one
+ * heads_as_rows != 0 (steps of single tokens over ONE kv head, G == 1, no talk / value_rot): every tile is one
  * token (count 1) and the 16 rows of a tensor-core tile are 16 consecutive query heads instead of 16 tokens, so a warp
  * serves 16 heads against the staged keys.  For b200_mixed_prompt_attn_splits such a step counts (H + 15) / 16 heads.
  * out_f32 as in b200_mixed_paged_attn_ext (not with value_rot). */
@@ -453,9 +453,7 @@ int b200_mixed_paged_attn_ext2(void* out, int64_t out_tok_stride, int64_t out_he
                                int chunk, int unrotate, int interleaved, float rot_base, int H, int G, int dk, int dv,
                                int v_row, int v_div, int out_f32, int block_size, int dtype, void* stream);
 
-/* b200_mixed_prompt_attn_ext with gate_per_channel as above (not with value_rot), and heads_as_rows for any number of kv heads:
- * the 16 rows of a tensor-core tile are up to 16 of the H / G query heads that share a kv head, with gates of either kind.  For
- * b200_mixed_prompt_attn_splits such a step counts G * ceil(H / G / 16) heads. */
+/* b200_mixed_prompt_attn_ext with gate_per_channel as above (not with value_rot); heads_as_rows goes with gates of either kind. */
 int b200_mixed_prompt_attn_ext2(void* out, int64_t out_tok_stride, int64_t out_head_stride, const void* q,
                                 int64_t q_tok_stride, int64_t q_head_stride, const void* gate, int64_t gate_stride,
                                 int gate_per_channel, const void* k_pool, const void* v_pool, const int32_t* block_tables,
@@ -465,8 +463,8 @@ int b200_mixed_prompt_attn_ext2(void* out, int64_t out_tok_stride, int64_t out_h
                                 int dv, int v_row, int v_div, int heads_as_rows, int out_f32, int block_size, int n_splits,
                                 float* workspace, int dtype, void* stream);
 
-/* Whether b200_mixed_prompt_attn_ext2 takes this layout with heads_as_rows (separate key and value pools). */
-int b200_mixed_prompt_attn_rows_supported(int H, int G, int dk, int dv, int dtype);
+/* Whether b200_mixed_prompt_attn_ext2 takes H heads over one kv head with heads_as_rows (separate key and value pools). */
+int b200_mixed_prompt_attn_rows_supported(int H, int dk, int dv, int dtype);
 
 /* b200_qknorm_rotary_append_ext with unit_norm: != 0: q and k rows are divided by their RMS even where q_norm / k_norm is NULL
  * (a norm without a weight: before or after the rotation is the same). */

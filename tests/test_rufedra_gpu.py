@@ -176,7 +176,7 @@ def _pages(k, v, bs, seed):
     return pools[0], pools[1], table.to(torch.int32)
 
 
-LAYOUTS = [(6, 2, 16, 16), (40, 2, 32, 24), (8, 8, 16, 8), (12, 4, 64, 64), (20, 1, 16, 64), (16, 2, 128, 128), (3, 1, 16, 8)]
+LAYOUTS = [(6, 2, 16, 16), (40, 2, 32, 24), (40, 1, 32, 24), (8, 8, 16, 8), (12, 4, 64, 64), (20, 1, 16, 64), (16, 2, 128, 128), (3, 1, 16, 8)]
 
 
 @pytest.mark.parametrize("H,G,dk,dv", LAYOUTS)
@@ -186,6 +186,8 @@ def test_attention_with_a_gate_per_channel_or_head(H, G, dk, dv, path, window):
     from dgi_b200 import mixer_ops as M
 
     kind, name = path.rsplit("-", 1)
+    if kind == "single-heads" and G > 1:
+        pytest.skip("heads go on the rows over one kv head")
     dt = {"fp32": torch.float32, "bf16": torch.bfloat16, "fp16": torch.float16}[name]
     g = torch.Generator().manual_seed(H * dk + dv)
     T, bs, scale = 333, 16, 1.0 / math.sqrt(dk)
@@ -227,7 +229,7 @@ def test_attention_with_a_gate_per_channel_or_head(H, G, dk, dv, path, window):
                 else:
                     tiles = [(i, min(16, n - i), 0) for i in range(0, n, 16)]
                 if kind == "single-heads":
-                    assert M.heads_as_rows_supported(H, G, dk, dv, dt)
+                    assert M.heads_as_rows_supported(H, dk, dv, dt)
                 for ctx in (0, 333):                                  # one CTA per tile, and the keys divided over several
                     M.mixed_prompt_attention(view, q.to(DEV), kp, vp, tables, torch.tensor(tiles, dtype=torch.int32, device=DEV),
                                              tp, scale, max_context=ctx, heads_as_rows=kind == "single-heads", **kw)
