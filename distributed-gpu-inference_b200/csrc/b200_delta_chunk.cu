@@ -856,7 +856,8 @@ int b200_delta_chunk_scan(float* o_raw, const void* q, const void* k, const void
   else run(delta_prepare_kernel<256>, prepare_smem<256>(), pg, 128);
   if (const int rc = check_launch("b200_delta_chunk_scan (prepare)")) return rc;
   auto scan = [&](auto kern, size_t smem, int dvb, int nt) { run(kern, smem, dim3(n_seqs, H, (dv + dvb - 1) / dvb), nt); };
-  const bool narrow = dv <= 32;
+  // blocks of 32 value columns also where blocks of 64 would leave SMs idle: the walk is a chain, and theirs is shorter
+  const bool narrow = dv <= 32 || static_cast<int64_t>(n_seqs) * H * ((dv + 63) / 64) <= kNumSMs;
   if (dk <= 64) {
     if (narrow) scan(delta_chunk_scan_kernel<64, 32, 1>, DeltaShape<64, 32, 1>::kBytes, 32, 128);
     else scan(delta_chunk_scan_kernel<64, 64, 1>, DeltaShape<64, 64, 1>::kBytes, 64, 128);

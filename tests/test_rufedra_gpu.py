@@ -268,7 +268,8 @@ def _delta_run(M, x, z, dt_bias, a_log, state, seqs, H, G, dk, dv, max_count):
 
 
 DELTAS = [(6, 3, 6, 10), (3, 1, 33, 3), (4, 2, 32, 48), (2, 2, 128, 64), (2, 1, 160, 24), (1, 1, 1, 1), (4, 4, 64, 128), (2, 1, 256, 100),
-          (8, 2, 128, 32), (2, 2, 72, 40)]
+          (8, 2, 128, 32), (2, 2, 72, 40),
+          (76, 2, 20, 40), (80, 1, 128, 72), (75, 75, 130, 64)]      # enough heads for the widest blocks of value columns
 
 
 @pytest.mark.parametrize("H,G,dk,dv", DELTAS)
