@@ -3,7 +3,7 @@
 //   sandwich residual        x += s * ls * w * y * rsqrt(mean(y^2) + eps);  out = w_next * x * rsqrt(mean(x^2) + eps_next): the
 //                            post-norm of one sublayer and the pre-norm of the next in one pass over the row
 //   gated linear unit        gelu_tanh(g) * u
-//   selective scan           per channel c and state n, with dt = softplus(z + bias) and A = -exp(A_log):
+//   selective scan           per channel c and state n, with dt = softplus(z + bias) and rates A < 0:
 //                              S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n;   y_c = sum_n S[c, n] C_n + D_c x_c
 //                            and out = gain * y * silu(gate), for portions of any length or one token per sequence
 //
@@ -223,7 +223,7 @@ struct SelArgs {
   const void* x; int64_t x_stride;
   const void* dt; int64_t dt_stride;
   const float* dt_bias;
-  const float* a_log;                 // [I][N]
+  const float* a;                     // [I][N], the rates
   const void* b; const void* c; int64_t bc_stride;
   const float* skip;                  // [I]
   const void* z; int64_t z_stride;
@@ -391,7 +391,7 @@ selective_scan_kernel(const SelArgs A) {
       const int n = sub * NPT + j + i;
       const bool ok = has && n < N;
       s[i] = (ok && !sq.fresh) ? st[n] : 0.f;
-      a[i] = ok ? -expf(A.a_log[static_cast<int64_t>(ch) * N + n]) * (sizeof(T) == 4 ? 1.0f : 1.4426950408889634f) : 0.f;
+      a[i] = ok ? A.a[static_cast<int64_t>(ch) * N + n] * (sizeof(T) == 4 ? 1.0f : 1.4426950408889634f) : 0.f;
     }
     S[j / 2] = pack2(s[0], s[1]);
     a2[j / 2] = pack2(a[0], a[1]);
@@ -513,56 +513,95 @@ selective_scan_kernel(const SelArgs A) {
   }
 }
 
-// One token per sequence: bound by the state's bytes, which are read and written once, in 16-byte pieces when V = 4.
-template <typename T, int V>
+// One token per sequence: bound by the state's bytes, which are read and written once, in 16-byte pieces when V = 4.  A thread
+// asks memory for everything it needs - P pieces of a channel's state among it - before it computes.
+template <typename T, int V, int P>
 __global__ void __launch_bounds__(128)
 selective_step_kernel(const SelArgs A) {
   const SelSeq sq = A.seqs[blockIdx.y];
   const int lg = A.lg, L = 1 << lg, N = A.N;
   const int ch = blockIdx.x * (128 >> lg) + (threadIdx.x >> lg), sub = threadIdx.x & (L - 1);
-  const bool has = ch < A.I;
+  const bool has = ch < A.I, writes = has && sub == 0;
   const int64_t n = sq.tok0;
-  float y = 0.f, x = 0.f;
+  float y = 0.f, x = 0.f, z = 0.f, skip = 0.f;
   if (has) {
-    x = Cvt<T>::to_f32(static_cast<const T*>(A.x)[n * A.x_stride + ch]);
-    const float dt = softplus_f(Cvt<T>::to_f32(static_cast<const T*>(A.dt)[n * A.dt_stride + ch]) + A.dt_bias[ch]);
-    const float dx = dt * x;
+    float* st = A.state + (static_cast<int64_t>(sq.slot) * A.I + ch) * N;
+    const float* al = A.a + static_cast<int64_t>(ch) * N;
     const T* bp = static_cast<const T*>(A.b) + n * A.bc_stride;
     const T* cp = static_cast<const T*>(A.c) + n * A.bc_stride;
-    float* st = A.state + (static_cast<int64_t>(sq.slot) * A.I + ch) * N;
-    const float* al = A.a_log + static_cast<int64_t>(ch) * N;
-    for (int i = sub * V; i < N; i += L * V) {
-      float s[V], a[V];
+    float s[P][V], a[P][V], bb[P][V], cc[P][V];
+    auto fetch = [&](int p, int i) {
       if constexpr (V == 4) {
         const float4 r = *reinterpret_cast<const float4*>(al + i);
-        a[0] = r.x; a[1] = r.y; a[2] = r.z; a[3] = r.w;
+        a[p][0] = r.x; a[p][1] = r.y; a[p][2] = r.z; a[p][3] = r.w;
         const float4 q = sq.fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(st + i);
-        s[0] = q.x; s[1] = q.y; s[2] = q.z; s[3] = q.w;
+        s[p][0] = q.x; s[p][1] = q.y; s[p][2] = q.z; s[p][3] = q.w;
       } else {
-        a[0] = al[i];
-        s[0] = sq.fresh ? 0.f : st[i];
+        a[p][0] = al[i];
+        s[p][0] = sq.fresh ? 0.f : st[i];
       }
+      if (V == 4 && A.vec_bc) {
+        struct alignas(V * sizeof(T)) Four { T e[V]; };
+        const Four b4 = *reinterpret_cast<const Four*>(bp + i), c4 = *reinterpret_cast<const Four*>(cp + i);
 #pragma unroll
-      for (int u = 0; u < V; ++u) {
-        s[u] += fmaf(expm1f(-expf(a[u]) * dt), s[u], dx * Cvt<T>::to_f32(bp[i + u]));
-        y = fmaf(s[u], Cvt<T>::to_f32(cp[i + u]), y);
+        for (int u = 0; u < V; ++u) {
+          bb[p][u] = Cvt<T>::to_f32(b4.e[u]);
+          cc[p][u] = Cvt<T>::to_f32(c4.e[u]);
+        }
+      } else {
+#pragma unroll
+        for (int u = 0; u < V; ++u) {
+          bb[p][u] = Cvt<T>::to_f32(bp[i + u]);
+          cc[p][u] = Cvt<T>::to_f32(cp[i + u]);
+        }
       }
-      if constexpr (V == 4) *reinterpret_cast<float4*>(st + i) = make_float4(s[0], s[1], s[2], s[3]);
-      else st[i] = s[0];
+    };
+    int i0 = sub * V;
+#pragma unroll
+    for (int p = 0; p < P; ++p)
+      if (i0 + p * L * V < N) fetch(p, i0 + p * L * V);
+    x = Cvt<T>::to_f32(static_cast<const T*>(A.x)[n * A.x_stride + ch]);
+    if (writes) {
+      z = Cvt<T>::to_f32(static_cast<const T*>(A.z)[n * A.z_stride + ch]);
+      skip = A.skip[ch];
+    }
+    const float dt = step_of<T>(Cvt<T>::to_f32(static_cast<const T*>(A.dt)[n * A.dt_stride + ch]) + A.dt_bias[ch]);
+    const float dx = dt * x, dts = sizeof(T) == 4 ? dt : dt * 1.4426950408889634f;    // 16-bit models: powers of two
+    while (i0 < N) {
+#pragma unroll
+      for (int p = 0; p < P; ++p) {
+        const int i = i0 + p * L * V;
+        if (i >= N) continue;
+        if constexpr (V == 4) {
+          const f32x2 dt2 = pack2(dts, dts), dx2 = pack2(dx, dx);
+#pragma unroll
+          for (int u = 0; u < V; u += 2)
+            unpack2(decayed<T>(pack2(s[p][u], s[p][u + 1]), dt2, pack2(a[p][u], a[p][u + 1]),
+                               mul2(dx2, pack2(bb[p][u], bb[p][u + 1]))), s[p][u], s[p][u + 1]);
+          *reinterpret_cast<float4*>(st + i) = make_float4(s[p][0], s[p][1], s[p][2], s[p][3]);
+        } else {
+          float unused;
+          unpack2(decayed<T>(pack2(s[p][0], 0.f), pack2(dts, 0.f), pack2(a[p][0], 0.f), pack2(dx * bb[p][0], 0.f)), s[p][0], unused);
+          st[i] = s[p][0];
+        }
+#pragma unroll
+        for (int u = 0; u < V; ++u) y = fmaf(s[p][u], cc[p][u], y);
+      }
+      i0 += P * L * V;
+#pragma unroll
+      for (int p = 0; p < P; ++p)
+        if (i0 + p * L * V < N) fetch(p, i0 + p * L * V);
     }
   }
   for (int o = 1; o < L; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
-  if (has && sub == 0) {
-    y = fmaf(A.skip[ch], x, y);
-    const float z = Cvt<T>::to_f32(static_cast<const T*>(A.z)[n * A.z_stride + ch]);
-    static_cast<T*>(A.out)[n * A.out_stride + ch] = Cvt<T>::from_f32(A.gain * y * silu_f(z));
-  }
+  if (writes)
+    static_cast<T*>(A.out)[n * A.out_stride + ch] = Cvt<T>::from_f32(A.gain * fmaf(skip, x, y) * gate_of<T>(z));
 }
 
 inline int sel_check(const char* what, const SelArgs& A, int n_seqs) {
   if (n_seqs < 0 || A.I <= 0 || A.N <= 0) return fail(B200_EINVAL, "%s: bad sizes", what);
   if (n_seqs > 65535) return fail(B200_ESHAPE, "%s: %d sequences", what, n_seqs);
-  if (n_seqs > 0 && (!A.out || !A.x || !A.dt || !A.dt_bias || !A.a_log || !A.b || !A.c || !A.skip || !A.z || !A.state || !A.seqs))
+  if (n_seqs > 0 && (!A.out || !A.x || !A.dt || !A.dt_bias || !A.a || !A.b || !A.c || !A.skip || !A.z || !A.state || !A.seqs))
     return fail(B200_EINVAL, "%s: null pointer", what);
   return 0;
 }
@@ -624,10 +663,10 @@ int b200_gelu_glu(void* y, const void* gu, int64_t rows, int ff, int dtype, void
 }
 
 int b200_selective_scan(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* dt, int64_t dt_stride,
-                        const float* dt_bias, const float* a_log, const void* b, const void* c, int64_t bc_stride,
+                        const float* dt_bias, const float* a, const void* b, const void* c, int64_t bc_stride,
                         const float* skip, const void* z, int64_t z_stride, float gain, float* state, const int32_t* seqs,
                         int n_seqs, int inner, int n_state, int dtype, void* stream) {
-  SelArgs A{out, out_stride, x, x_stride, dt, dt_stride, dt_bias, a_log, b, c, bc_stride, skip, z, z_stride, gain, state,
+  SelArgs A{out, out_stride, x, x_stride, dt, dt_stride, dt_bias, a, b, c, bc_stride, skip, z, z_stride, gain, state,
             reinterpret_cast<const SelSeq*>(seqs), inner, n_state, 0, 0, 0};
   if (const int rc = sel_check("b200_selective_scan", A, n_seqs)) return rc;
   if (n_state > 256) return fail(B200_ESHAPE, "b200_selective_scan: %d states per channel beyond 256", n_state);
@@ -660,22 +699,25 @@ int b200_selective_scan(void* out, int64_t out_stride, const void* x, int64_t x_
 }
 
 int b200_selective_step(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* dt, int64_t dt_stride,
-                        const float* dt_bias, const float* a_log, const void* b, const void* c, int64_t bc_stride,
+                        const float* dt_bias, const float* a, const void* b, const void* c, int64_t bc_stride,
                         const float* skip, const void* z, int64_t z_stride, float gain, float* state, const int32_t* seqs,
                         int n_seqs, int inner, int n_state, int dtype, void* stream) {
-  SelArgs A{out, out_stride, x, x_stride, dt, dt_stride, dt_bias, a_log, b, c, bc_stride, skip, z, z_stride, gain, state,
+  SelArgs A{out, out_stride, x, x_stride, dt, dt_stride, dt_bias, a, b, c, bc_stride, skip, z, z_stride, gain, state,
             reinterpret_cast<const SelSeq*>(seqs), inner, n_state, 0, 0, 0};
   if (const int rc = sel_check("b200_selective_step", A, n_seqs)) return rc;
   if (n_seqs == 0) return 0;
   const int per = n_state % 4 == 0 ? n_state / 4 : n_state;      // pieces of a channel's state
-  while (A.lg < 5 && (1 << A.lg) < per) ++A.lg;
+  const int pieces = per > 1 ? 2 : 1;                            // per lane at a time
+  while (A.lg < 5 && (pieces << A.lg) < per) ++A.lg;
   const int ch = 128 >> A.lg;
   return selective_by_dtype(dtype, "b200_selective_step", [&](auto* tag) {
     using T = std::remove_pointer_t<decltype(tag)>;
+    A.vec_bc = bc_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(b) | reinterpret_cast<uintptr_t>(c)) % (4 * sizeof(T)) == 0;
     const dim3 grid((inner + ch - 1) / ch, n_seqs);
     auto s = static_cast<cudaStream_t>(stream);
-    if (n_state % 4 == 0) selective_step_kernel<T, 4><<<grid, 128, 0, s>>>(A);
-    else selective_step_kernel<T, 1><<<grid, 128, 0, s>>>(A);
+    if (n_state % 4 == 0 && pieces == 2) selective_step_kernel<T, 4, 2><<<grid, 128, 0, s>>>(A);
+    else if (n_state % 4 == 0) selective_step_kernel<T, 4, 1><<<grid, 128, 0, s>>>(A);
+    else selective_step_kernel<T, 1, 2><<<grid, 128, 0, s>>>(A);
     return check_launch("b200_selective_step");
   });
 }

@@ -1225,12 +1225,12 @@ def gated_part_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, eps:
 # ---- per-channel selective state spaces, sublayers normed on both sides (csrc/b200_selective_ops.cu) --------------------
 @_timed
 def selective_scan(x: torch.Tensor, dt: torch.Tensor, B: torch.Tensor, C: torch.Tensor, z: torch.Tensor, dt_bias: torch.Tensor,
-                   a_log: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, seqs: torch.Tensor, gain: float = 1.0,
+                   rates: torch.Tensor, skip: torch.Tensor, state: torch.Tensor, seqs: torch.Tensor, gain: float = 1.0,
                    out: Optional[torch.Tensor] = None, max_count: int = 0) -> torch.Tensor:
-    """Per channel ``c`` and state ``n``, with ``dt = softplus(dt + dt_bias)``: ``S <- e^(-e^a_log dt) S + dt x B``, ``y = S.C +
+    """Per channel ``c`` and state ``n``, with ``dt = softplus(dt + dt_bias)``: ``S <- e^(rate dt) S + dt x B``, ``y = S.C +
     skip x``; returns ``gain * y * silu(z)`` ``[n, inner]`` in the activations' dtype (``out`` may be a column slice of a wider
     buffer).  ``x / dt / z [n, inner]`` and ``B / C [n, N]`` (one row stride) may be column slices; ``dt_bias``, ``skip`` fp32
-    ``[inner]``, ``a_log`` fp32 ``[inner, N]``, ``state`` fp32 ``[slots, inner, N]``.  ``max_count``: the largest token count in
+    ``[inner]``, ``rates`` (negative) fp32 ``[inner, N]``, ``state`` fp32 ``[slots, inner, N]``.  ``max_count``: the largest token count in
     ``seqs``; steps of single tokens take a launch of their own."""
     _need_cuda(x, dt, B, C, z, state, seqs)
     _check_seqs(seqs)
@@ -1242,7 +1242,7 @@ def selective_scan(x: torch.Tensor, dt: torch.Tensor, B: torch.Tensor, C: torch.
         raise ValueError("B and C must share a row stride")
     if any(t.dtype != x.dtype for t in (dt, B, C, z)):
         raise TypeError("activations share one dtype")
-    for t, shape in ((dt_bias, (inner,)), (skip, (inner,)), (a_log, (inner, N)), (state, (state.shape[0], inner, N))):
+    for t, shape in ((dt_bias, (inner,)), (skip, (inner,)), (rates, (inner, N)), (state, (state.shape[0], inner, N))):
         if t.dtype != torch.float32 or tuple(t.shape) != shape or not t.is_contiguous():
             raise ValueError("constants and state are contiguous fp32")
     if out is None:
@@ -1251,7 +1251,7 @@ def selective_scan(x: torch.Tensor, dt: torch.Tensor, B: torch.Tensor, C: torch.
         raise ValueError("out must be [n, inner] in the activations' dtype")
     step = max_count == 1 and seqs.shape[0] == n
     fn = _lib_().b200_selective_step if step else _lib_().b200_selective_scan
-    rc = fn(out.data_ptr(), _rows2(out), x.data_ptr(), _rows2(x), dt.data_ptr(), _rows2(dt), dt_bias.data_ptr(), a_log.data_ptr(),
+    rc = fn(out.data_ptr(), _rows2(out), x.data_ptr(), _rows2(x), dt.data_ptr(), _rows2(dt), dt_bias.data_ptr(), rates.data_ptr(),
             B.data_ptr(), C.data_ptr(), _rows2(B), skip.data_ptr(), z.data_ptr(), _rows2(z), float(gain), state.data_ptr(),
             seqs.data_ptr(), seqs.shape[0], inner, N, DTYPE_ID[x.dtype], _stream())
     _lib.check_mixers(rc, "b200_selective_step" if step else "b200_selective_scan")

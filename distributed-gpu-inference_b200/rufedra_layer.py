@@ -169,7 +169,8 @@ class KeyValueSelectiveMixer(nn.Module):
                                        device, dtype)
         self.w_dt = _param(rt["dt"], device, dtype)
         f32 = lambda name: _param(rt[name], device, torch.float32)  # noqa: E731
-        self.dt_bias, self.a_log, self.skip = f32("dt.b"), f32("A_log"), f32("D")
+        self.dt_bias, self.skip = f32("dt.b"), f32("D")
+        self.rates = _param(-torch.exp(rt["A_log"].to(torch.float64)), device, torch.float32)
         # the two output projections side by side; the branch weights are folded as the module docstring says
         a_l, a_r = float(spec["left_scale"]), float(spec["right_scale"])
         c = a_l if a_l != 0.0 else 1.0
@@ -214,7 +215,7 @@ class KeyValueSelectiveMixer(nn.Module):
         p = F.linear(x, self.w_x)
         dt = F.linear(p[:, :self.rank], self.w_dt)
         mixer_ops.selective_scan(x, dt, p[:, x_cuts[1]:x_cuts[1] + N], p[:, x_cuts[2]:x_cuts[2] + N],
-                                 proj[:, c[4]:c[4] + inner], self.dt_bias, self.a_log, self.skip, state, st.scan_seqs,
+                                 proj[:, c[4]:c[4] + inner], self.dt_bias, self.rates, self.skip, state, st.scan_seqs,
                                  gain=self.right_gain, out=buf[:, self.right_at:self.right_at + inner],
                                  max_count=st.max_count())
         return F.linear(buf, self.w_out)

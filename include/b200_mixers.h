@@ -501,18 +501,18 @@ int b200_delta_step(float* o_raw, const void* q, const void* k, const void* v, i
                     int dtype, void* stream);
 
 /* Selective state space per (sequence, channel c) over the sequence's tokens of this step, in order (SeqSpan rows):
- *   dt = softplus(dt_logit + dt_bias);  S[c, n] <- exp(-exp(a_log[c, n]) dt_c) S[c, n] + dt_c x_c B_n;
+ *   dt = softplus(dt_logit + dt_bias);  S[c, n] <- exp(a[c, n] dt_c) S[c, n] + dt_c x_c B_n;
  *   out_c = gain * (sum_n S[c, n] C_n + skip_c x_c) * silu(z_c)
- * x, dt, z: T rows of `inner`; b, c: T rows of n_state with one row stride; out T rows; dt_bias, skip fp32 [inner]; a_log fp32
- * [inner, n_state]; state fp32 [slots, inner, n_state], read unless the sequence is fresh and written back.  n_state <= 256. */
+ * x, dt, z: T rows of `inner`; b, c: T rows of n_state with one row stride; out T rows; dt_bias, skip fp32 [inner]; a fp32
+ * [inner, n_state] (negative rates); state fp32 [slots, inner, n_state], read unless the sequence is fresh and written back.  n_state <= 256. */
 int b200_selective_scan(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* dt, int64_t dt_stride,
-                        const float* dt_bias, const float* a_log, const void* b, const void* c, int64_t bc_stride,
+                        const float* dt_bias, const float* a, const void* b, const void* c, int64_t bc_stride,
                         const float* skip, const void* z, int64_t z_stride, float gain, float* state, const int32_t* seqs,
                         int n_seqs, int inner, int n_state, int dtype, void* stream);
 
 /* The same for steps whose sequences bring ONE token each (any n_state). */
 int b200_selective_step(void* out, int64_t out_stride, const void* x, int64_t x_stride, const void* dt, int64_t dt_stride,
-                        const float* dt_bias, const float* a_log, const void* b, const void* c, int64_t bc_stride,
+                        const float* dt_bias, const float* a, const void* b, const void* c, int64_t bc_stride,
                         const float* skip, const void* z, int64_t z_stride, float gain, float* state, const int32_t* seqs,
                         int n_seqs, int inner, int n_state, int dtype, void* stream);
 

@@ -353,7 +353,7 @@ def test_selective_scan_over_portions_slots_and_single_tokens(inner, N, dt, tol,
     want = 0.7 * y * R.silu(z.to(F64))
     state = torch.full((3, inner, N), float("nan"), device=DEV)
     dw, dbc = wide.to(DEV), bc.to(DEV)
-    consts = [t.to(DEV) for t in (bias, a_log, D)]
+    consts = [t.to(DEV) for t in (bias, -torch.exp(a_log), D)]
     out = torch.full((n + 3, inner + 6), 9.0, dtype=dt, device=DEV)
     at = 0
     for cut in (70, 1, 1, 2, 33, 32, 31, 30):
@@ -375,6 +375,30 @@ def test_selective_scan_over_portions_slots_and_single_tokens(inner, N, dt, tol,
     assert torch.isnan(state[1]).all()
 
 
+@pytest.mark.parametrize("inner,N", [(520, 16), (515, 3), (1030, 12), (300, 136)])
+@pytest.mark.parametrize("dt,tol", [(torch.float32, 1e-5), (torch.bfloat16, 1e-2)], ids=["fp32", "bf16"])
+def test_selective_steps_of_many_sequences(inner, N, dt, tol):
+    """Slots in reverse, every third sequence fresh."""
+    from dgi_b200 import mixer_ops as M
+
+    g = torch.Generator().manual_seed(inner)
+    n = 230
+    x, dtl, z = (torch.randn(n, inner, generator=g).to(dt) for _ in range(3))
+    B, C = torch.randn(n, N, generator=g).to(dt), torch.randn(n, N, generator=g).to(dt)
+    bias, rates, D = torch.randn(inner, generator=g) - 1.0, -torch.rand(inner, N, generator=g), torch.randn(inner, generator=g)
+    fresh = torch.arange(n) % 3 == 0
+    state = torch.randn(n, inner, N, generator=g)
+    S = state.flip(0).to(F64) * (~fresh)[:, None, None]
+    step = R.softplus(dtl.to(F64) + bias.to(F64))
+    S = torch.exp(step[:, :, None] * rates.to(F64)) * S + (step * x.to(F64))[:, :, None] * B.to(F64)[:, None, :]
+    want = ((S * C.to(F64)[:, None, :]).sum(-1) + D.to(F64) * x.to(F64)) * R.silu(z.to(F64))
+    dev = state.to(DEV)
+    spans = seqs_of([(i, 1, n - 1 - i, int(fresh[i])) for i in range(n)])
+    out = M.selective_scan(*(t.to(DEV) for t in (x, dtl, B, C, z, bias, rates, D)), dev, spans, max_count=1)
+    close(out.cpu(), want, tol)
+    close(dev.cpu().flip(0), S, 1e-5)
+
+
 def test_selective_state_keeps_32_bit_accuracy_over_thousands_of_slow_tokens():
     from dgi_b200 import mixer_ops as M
 
@@ -384,7 +408,7 @@ def test_selective_state_keeps_32_bit_accuracy_over_thousands_of_slow_tokens():
     bias, a_log, D = torch.full((inner,), -5.0), torch.full((inner, N), -3.0), torch.zeros(inner)
     y, S = R.selective_scan(x.to(F64), R.softplus(dtl.to(F64) - 5.0), -torch.exp(a_log.to(F64)), B.to(F64), C.to(F64), D.to(F64))
     state = torch.zeros(1, inner, N, device=DEV)
-    out = M.selective_scan(*(t.to(DEV) for t in (x, dtl, B, C, z, bias, a_log, D)), state, seqs_of([(0, n, 0, 1)]), max_count=n)
+    out = M.selective_scan(*(t.to(DEV) for t in (x, dtl, B, C, z, bias, -torch.exp(a_log), D)), state, seqs_of([(0, n, 0, 1)]), max_count=n)
     close(out.cpu(), y * R.silu(z.to(F64)), 4e-6)
     close(state[0].cpu(), S, 4e-6)
 
